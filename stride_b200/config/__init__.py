@@ -5,6 +5,7 @@ from . import keralorn as _keralorn      # registers Keralorn
 from . import ganupel as _ganupel        # registers Ganupel
 from . import pusisun as _pusisun        # registers Pusisun
 from . import sitivik as _sitivik        # registers Sitivik
+from . import viperax as _viperax        # registers Viperax
 
 __all__ = ["ConfigError", "LlamaConfig", "RopeScaling", "Architecture", "register_architecture",
            "registered_architectures", "resolve_architecture"]

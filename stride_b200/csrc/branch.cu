@@ -264,15 +264,15 @@ SB_EXPORT int sb_row_scaled_add(float* dst, const void* x, int x_dtype, const fl
 
 // ------------------------------------------------------------------ operations of the native step program (step_ops.h)
 // i: 0 dst, 1 a, 2 a's partial sums (flat), 3 their K ranges S, 4 most tokens with a buffer per range, 5 b, 6 b's partial sums, 7 their S,
-//    8 gain, 9 gain dtype, 10 W
+//    8 gain, 9 gain dtype, 10 W, 11 a limit of a's own in place of i[4] (or 0), 12 the same for b
 // f: 0 ca, 1 cb
 SB_EXPORT int sb_op_branch_fold(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
   const int W = (int)op->i[10];
   const int64_t stride = static_cast<int64_t>(s->n) * W;
-  return sb_branch_fold(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[4], s->n), stride,
-                        static_cast<float>(op->f[0]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]), partial_count(op->i[7], op->i[4], s->n),
+  return sb_branch_fold(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
+                        static_cast<float>(op->f[0]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]), partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n),
                         stride, static_cast<float>(op->f[1]), ptr<const void>(op->i[8]), (int)op->i[9], s->n, W, static_cast<cudaStream_t>(stream));
 }
 
@@ -282,8 +282,8 @@ SB_EXPORT int sb_op_branch_norm_fold(const SbOp* op, const SbStep* s, void* stre
   if (s->n <= 0) return SB_OP_SKIPPED;
   const int W = (int)op->i[10];
   const int64_t stride = static_cast<int64_t>(s->n) * W;
-  return sb_branch_norm_fold(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[4], s->n), stride,
-                             static_cast<float>(op->f[0]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]), partial_count(op->i[7], op->i[4], s->n),
+  return sb_branch_norm_fold(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
+                             static_cast<float>(op->f[0]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]), partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n),
                              stride, static_cast<float>(op->f[1]), ptr<const void>(op->i[8]), (int)op->i[9], static_cast<float>(op->f[2]), s->n, W,
                              static_cast<cudaStream_t>(stream));
 }
@@ -400,4 +400,26 @@ SB_EXPORT int sb_op_branch_pair_norm_fold(const SbOp* op, const SbStep* s, void*
   }
 #undef SB_PAIR
   return sb::check_launch("sb_op_branch_pair_norm_fold");
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------------
+// A branch buffer set to zero, for an operation that adds to a branch nothing was stored into yet.
+namespace {
+
+__global__ void __launch_bounds__(256) branch_clear_kernel(float* __restrict__ dst, int64_t total) {
+  sb::grid_launch_dependents();
+  sb::grid_dependency_wait();
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * blockDim.x)
+    dst[i] = 0.0f;
+}
+
+}  // namespace
+
+// i: 0 dst, 1 W
+SB_EXPORT int sb_op_branch_clear(const SbOp* op, const SbStep* s, void* stream) {
+  if (s->n <= 0) return SB_OP_SKIPPED;
+  const int64_t total = static_cast<int64_t>(s->n) * op->i[1], blocks = (total + 255) / 256, most = 8ll * sb::sm_count();
+  sb::launch_pdl(branch_clear_kernel, dim3(static_cast<unsigned>(blocks < most ? blocks : most)), dim3(256), 0, static_cast<cudaStream_t>(stream),
+                 sbstep::ptr<float>(op->i[0]), total);
+  return sb::check_launch("sb_op_branch_clear");
 }

@@ -545,3 +545,44 @@ SB_EXPORT int sb_op_cast_columns(const SbOp* op, const SbStep* s, void* stream) 
   else return sb::fail("sb_op_cast_columns: unsupported dtype %d", (int)op->i[7]), SB_OP_FAILED;
   return sb::check_launch("sb_op_cast_columns");
 }
+
+// ------------------------------------------------------------------ logits
+// logits <- cap tanh(scale logits / cap) in place (cap 0: scale alone), on the rows whose logits are wanted; 32-bit.
+namespace {
+
+__device__ __forceinline__ float capped(float v, float scale, float cap) {
+  v = __fmul_rn(v, scale);
+  return cap > 0.0f ? __fmul_rn(cap, tanhf(v / cap)) : v;
+}
+
+__global__ void __launch_bounds__(256) cap_logits_kernel(float* __restrict__ logits, int64_t total, float scale, float cap, int vec) {
+  sb::grid_launch_dependents();
+  sb::grid_dependency_wait();
+  const int64_t step = static_cast<int64_t>(gridDim.x) * blockDim.x, at = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (vec) {
+    float4* l4 = reinterpret_cast<float4*>(logits);
+    for (int64_t i = at; i < total / 4; i += step) {
+      const float4 v = l4[i];
+      l4[i] = make_float4(capped(v.x, scale, cap), capped(v.y, scale, cap), capped(v.z, scale, cap), capped(v.w, scale, cap));
+    }
+  } else {
+    for (int64_t i = at; i < total; i += step) logits[i] = capped(logits[i], scale, cap);
+  }
+}
+
+}  // namespace
+
+SB_EXPORT int sb_cap_logits(float* logits, int64_t total, float scale, float cap, cudaStream_t stream) {
+  if (total <= 0) return 0;
+  const int vec = total % 4 == 0 && (reinterpret_cast<uintptr_t>(logits) & 15) == 0;
+  const int64_t blocks = (total / (vec ? 4 : 1) + 255) / 256, most = 16ll * sb::sm_count();
+  sb::launch_pdl(cap_logits_kernel, dim3(static_cast<unsigned>(blocks < most ? blocks : most)), dim3(256), 0, stream, logits, total, scale, cap, vec);
+  return sb::check_launch("sb_cap_logits");
+}
+
+// i: 0 logits [wanted][vocab] float32, 1 vocab      f: 0 scale, 1 cap (0: none)
+SB_EXPORT int sb_op_cap_logits(const SbOp* op, const SbStep* s, void* stream) {
+  if (s->wanted <= 0) return SB_OP_SKIPPED;
+  return sb_cap_logits(sbstep::ptr<float>(op->i[0]), static_cast<int64_t>(s->wanted) * op->i[1], (float)op->f[0], (float)op->f[1],
+                       static_cast<cudaStream_t>(stream));
+}

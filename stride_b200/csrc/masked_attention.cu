@@ -11,8 +11,10 @@
 //
 // Kernels in front prepare a step's tokens: `qkv_norm_append_kernel` (bias, an RMS norm over the whole query projection and
 // over the whole key projection, append), `latent_prepare_kernel` (the two latents of latent attention normed, the shared rotated key
-// part, append of one row per token), `rotate_heads_kernel` (rotation of a slice of every query head) and `head_linear_kernel` (a
-// matrix per head: the key projection taken into the queries in front of the attention, the value projection behind it).
+// part, append of one row per token), `latent_direct_kernel` (the same for queries without a latent: stored as projected; the key/value
+// latent normed and appended, or left out by layers that read another layer's), `rotate_heads_kernel` (rotation of a slice of every query
+// head) and `head_linear_kernel` (a matrix per head: the key projection taken into the queries in front of the attention, the value
+// projection behind it, there with a sigmoid gate per element on the way out where a design has one).
 #include "common.cuh"
 #include "step_ops.h"
 
@@ -160,6 +162,96 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(LatentParams p) {
   }
 }
 
+struct DirectParams {
+  const float* proj;         // [P][n][width]: the queries (Q elements), the key/value latent (R; none for a layer that stores none), then
+                             // whatever else the projection carries
+  int n_partials;
+  int64_t partial_stride;
+  int width;
+  const float* kv_gain;      // [R]
+  float eps;
+  const int32_t* positions;
+  const int32_t* slots;
+  void* q_out;               // [n][Q]
+  PageRef c;                 // one row per token: the latent
+  int Q, R;
+};
+
+__device__ __forceinline__ float4 folded4(const float* p, int n_partials, int64_t stride) {
+  float4 part[kInFlight];
+#pragma unroll
+  for (int s = 0; s < kInFlight; ++s)
+    if (s < n_partials) part[s] = *reinterpret_cast<const float4*>(p + s * stride);
+  float4 sum = part[0];
+#pragma unroll
+  for (int s = 1; s < kInFlight; ++s)
+    if (s < n_partials) sum.x += part[s].x, sum.y += part[s].y, sum.z += part[s].z, sum.w += part[s].w;
+  for (int s = kInFlight; s < n_partials; ++s) {
+    const float4 a = *reinterpret_cast<const float4*>(p + s * stride);
+    sum.x += a.x, sum.y += a.y, sum.z += a.z, sum.w += a.w;
+  }
+  return sum;
+}
+__device__ __forceinline__ void store4(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store4(bf16* dst, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 packed;
+  packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+  packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(dst) = packed;
+}
+
+// A block per token (blockIdx.y 0: the latent, the further ones: shares of the queries): the queries as projected; the latent RMS-normed
+// with its gain and appended to the token's page. VEC: every size a multiple of four, four elements a thread and request.
+template <class T, bool VEC>
+__global__ void __launch_bounds__(128) latent_direct_kernel(DirectParams p) {
+  extern __shared__ __align__(16) float row_values[];
+  __shared__ float red[32];
+  constexpr int VE = VEC ? 4 : 1;
+  sb::grid_launch_dependents();
+  const int row = blockIdx.x, part = static_cast<int>(blockIdx.y) - (p.R > 0 ? 1 : 0);
+  int pos = 0, page = 0;
+  if (part < 0) {
+    pos = p.positions[row];
+    page = p.c.block_table[static_cast<int64_t>(p.slots[row]) * p.c.max_pages + pos / p.c.page_size];
+  }
+  sb::grid_dependency_wait();
+  const float* src = p.proj + static_cast<int64_t>(row) * p.width;
+  if (part >= 0) {
+    T* q = static_cast<T*>(p.q_out) + static_cast<int64_t>(row) * p.Q;
+    const int shares = static_cast<int>(gridDim.y) - (p.R > 0 ? 1 : 0);
+    for (int i = (part * blockDim.x + threadIdx.x) * VE; i < p.Q; i += shares * blockDim.x * VE) {
+      if constexpr (VEC) store4(q + i, folded4(src + i, p.n_partials, p.partial_stride));
+      else q[i] = sb::narrow<T>(folded(src + i, p.n_partials, p.partial_stride));
+    }
+    return;
+  }
+  src += p.Q;
+  float sq = 0.0f;
+  for (int i = threadIdx.x * VE; i < p.R; i += blockDim.x * VE) {
+    if constexpr (VEC) {
+      const float4 v = folded4(src + i, p.n_partials, p.partial_stride);
+      *reinterpret_cast<float4*>(row_values + i) = v;
+      sq = fmaf(v.x, v.x, sq), sq = fmaf(v.y, v.y, sq), sq = fmaf(v.z, v.z, sq), sq = fmaf(v.w, v.w, sq);
+    } else {
+      const float v = folded(src + i, p.n_partials, p.partial_stride);
+      row_values[i] = v;
+      sq = fmaf(v, v, sq);
+    }
+  }
+  const float r = 1.0f / sqrtf(sb::block_sum(sq, red) / static_cast<float>(p.R) + p.eps);
+  T* dst = static_cast<T*>(p.c.pages) + static_cast<int64_t>(page) * p.c.page_stride + static_cast<int64_t>(pos % p.c.page_size) * p.c.Dc;
+  for (int i = threadIdx.x * VE; i < p.R; i += blockDim.x * VE) {       // (a thread reads back what it wrote)
+    if constexpr (VEC) {
+      const float4 v = *reinterpret_cast<const float4*>(row_values + i), g = *reinterpret_cast<const float4*>(p.kv_gain + i);
+      store4(dst + i, make_float4(__fmul_rn(__fmul_rn(v.x, r), g.x), __fmul_rn(__fmul_rn(v.y, r), g.y), __fmul_rn(__fmul_rn(v.z, r), g.z),
+                                  __fmul_rn(__fmul_rn(v.w, r), g.w)));
+    } else {
+      dst[i] = sb::narrow<T>(__fmul_rn(__fmul_rn(row_values[i], r), p.kv_gain[i]));
+    }
+  }
+}
+
 // q [P][n][H D] partial sums -> out [n][H D]: elements offset .. offset + rot - 1 of every head rotated by the token's position, the
 // others passed on.
 template <class T>
@@ -190,7 +282,15 @@ struct HeadLinearParams {
   void* out;                 // row r, head h: out + r out_row + h out_head, N elements (and the tail behind them)
   int64_t out_row, out_head;
   int n, H, K, N, tail;
+  const float* gate;         // null, or partial sums [P][n][gate_width] whose element (r, h N + j) gates output j of head h: times its sigmoid
+  int gate_partials, gate_width;
+  int64_t gate_stride;
 };
+
+// The gate of output j of head h, row r; gates are partial sums of a projection like any other.
+__device__ __forceinline__ float head_gate(const HeadLinearParams& p, int r, int h, int j) {
+  return 1.0f / (1.0f + expf(-folded(p.gate + static_cast<int64_t>(r) * p.gate_width + h * p.N + j, p.gate_partials, p.gate_stride)));
+}
 
 // out[r, h, :N] = W_h^T in[r, h, :K], a matrix per head; the `tail` elements behind the K pass unchanged. A block is TR rows of one head: the
 // rows wait in shared memory, a thread owns output columns and walks K in ascending order, so a row's result does not depend on its
@@ -224,7 +324,8 @@ __global__ void __launch_bounds__(128) head_linear_kernel(HeadLinearParams p) {
     }
 #pragma unroll
     for (int r = 0; r < TR; ++r)
-      if (r0 + r < p.n) out[static_cast<int64_t>(r0 + r) * p.out_row + j] = sb::narrow<T>(acc[r]);
+      if (r0 + r < p.n)
+        out[static_cast<int64_t>(r0 + r) * p.out_row + j] = sb::narrow<T>(p.gate != nullptr ? acc[r] * head_gate(p, r0 + r, h, j) : acc[r]);
   }
 }
 
@@ -417,7 +518,11 @@ __global__ void __launch_bounds__(128) head_linear_tc_kernel(HeadLinearParams p)
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const int c = (i >> 1) * 16 + (i & 1) * 8;
-      if (n0 + c + (lane & 3) * 2 < p.N) *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(acc[i][2 * half], acc[i][2 * half + 1]);
+      const int j = n0 + c + (lane & 3) * 2;
+      if (j >= p.N) continue;
+      float a = acc[i][2 * half], b = acc[i][2 * half + 1];
+      if (p.gate != nullptr) a *= head_gate(p, r, h, j), b *= head_gate(p, r, h, j + 1);
+      *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(a, b);
     }
   }
 }
@@ -790,14 +895,17 @@ SB_EXPORT int sb_rotate_heads(const float* q, int n_partials, int64_t partial_st
 }
 
 // out[r, h, :N] = W_h^T in[r, h, :K] for every head (w [H][K][N]); `tail` elements behind the K are copied behind the N. Strides in elements.
-SB_EXPORT int sb_head_linear(const void* in, int64_t in_row, int64_t in_head, const void* w, void* out, int64_t out_row, int64_t out_head, int dtype,
-                             int n, int H, int K, int N, int tail, cudaStream_t stream) {
+// gate: null, or partial sums [P][n][gate_width]: output j of head h times the sigmoid of element (r, h N + j).
+SB_EXPORT int sb_head_linear_gated(const void* in, int64_t in_row, int64_t in_head, const void* w, void* out, int64_t out_row, int64_t out_head,
+                                   int dtype, int n, int H, int K, int N, int tail, const float* gate, int gate_partials, int64_t gate_stride,
+                                   int gate_width, cudaStream_t stream) {
   if (n <= 0) return 0;
+  if (gate != nullptr && (tail != 0 || gate_partials < 1)) return sb::fail("sb_head_linear: a gate goes with no tail and at least one partial sum");
   if (H <= 0 || K <= 0 || N <= 0 || tail < 0) return sb::fail("sb_head_linear: %d heads of %d -> %d (+ %d)", H, K, N, tail);
   constexpr int TR = 8;
   const size_t smem = sizeof(float) * TR * K;
   if (smem > 160 * 1024) return sb::fail("sb_head_linear: rows of %d elements do not fit the row buffer", K);
-  HeadLinearParams p{in, in_row, in_head, w, out, out_row, out_head, n, H, K, N, tail};
+  HeadLinearParams p{in, in_row, in_head, w, out, out_row, out_head, n, H, K, N, tail, gate, gate_partials, gate_width, gate_stride};
   const bool aligned = ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   if (dtype == 1 && aligned && K % 16 == 0 && N % 8 == 0 && in_row % 8 == 0 && in_head % 8 == 0 && out_row % 8 == 0 && out_head % 8 == 0) {
     // (what decides for the tensor cores is the shape alone, never the number of rows: a token has one form whatever step it is in)
@@ -815,6 +923,11 @@ SB_EXPORT int sb_head_linear(const void* in, int64_t in_row, int64_t in_head, co
     return sb::fail("sb_head_linear: unsupported dtype %d", dtype);
   }
   return sb::check_launch("sb_head_linear");
+}
+
+SB_EXPORT int sb_head_linear(const void* in, int64_t in_row, int64_t in_head, const void* w, void* out, int64_t out_row, int64_t out_head, int dtype,
+                             int n, int H, int K, int N, int tail, cudaStream_t stream) {
+  return sb_head_linear_gated(in, in_row, in_head, w, out, out_row, out_head, dtype, n, H, K, N, tail, nullptr, 0, 0, 0, stream);
 }
 
 // `chunk` > 0: a row sees only the keys of its own chunk of that many positions; `out_f32`: the result is stored as float32.
@@ -925,12 +1038,41 @@ SB_EXPORT int sb_op_rotate_heads(const SbOp* op, const SbStep* s, void* stream) 
                          static_cast<cudaStream_t>(stream));
 }
 
-// i: 0 in, 1 in_row, 2 in_head, 3 w, 4 out, 5 out_row, 6 out_head, 7 dtype, 8 H, 9 K, 10 N, 11 tail
+// i: 0 projection partial sums (flat), 1 their width, 2 K ranges S, 3 most tokens with a buffer per range, 4 kv gain, 5 q out, 6 dtype, 7 pages,
+//    8 block table, 9 max_pages, 10 page_size, 11 page_stride, 12 Q, 13 R (0: no latent is stored), 14 Dc      f: 0 eps
+SB_EXPORT int sb_op_latent_direct(const SbOp* op, const SbStep* s, void* stream) {
+  using namespace sbstep;
+  const int n = s->n, width = (int)op->i[1], Q = (int)op->i[12], R = (int)op->i[13], Dc = (int)op->i[14], dtype = (int)op->i[6];
+  if (n <= 0) return SB_OP_SKIPPED;
+  if (Q <= 0 || R < 0 || Q + R > width || (R > 0 && Dc < R)) return sb::fail("sb_op_latent_direct: %d queries and a latent of %d in rows of %d / %d", Q, R, width, Dc), SB_OP_FAILED;
+  if (dtype != 0 && dtype != 1) return sb::fail("sb_op_latent_direct: unsupported dtype %d", dtype), SB_OP_FAILED;
+  const size_t smem = static_cast<size_t>(R > 0 ? R : 1) * sizeof(float);
+  if (smem > 40 * 1024) return sb::fail("sb_op_latent_direct: a latent of %d elements does not fit the row buffer", R), SB_OP_FAILED;
+  DirectParams p{ptr<const float>(op->i[0]), partial_count(op->i[2], op->i[3], n), static_cast<int64_t>(n) * width, width, ptr<const float>(op->i[4]),
+                 (float)op->f[0], positions(s), slots(s), ptr<void>(op->i[5]),
+                 page_ref(ptr<void>(op->i[7]), ptr<const int32_t>(op->i[8]), (int)op->i[9], (int)op->i[10], op->i[11], 0, 0, Dc), Q, R};
+  // (which form runs depends on the sizes and the buffers alone, never on the rows of the step)
+  const bool vec = width % 4 == 0 && Q % 4 == 0 && R % 4 == 0 && Dc % 4 == 0 && op->i[11] % 4 == 0 &&
+                   ((op->i[0] | op->i[4] | op->i[5] | op->i[7]) & 15) == 0;
+  const int per_block = 128 * (vec ? 4 : 1) * 2;                    // queries: two requests a thread
+  const dim3 grid(n, (Q + per_block - 1) / per_block + (R > 0 ? 1 : 0));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dtype == 0 && vec) sb::launch_pdl(latent_direct_kernel<float, true>, grid, dim3(128), smem, st, p);
+  else if (dtype == 0) sb::launch_pdl(latent_direct_kernel<float, false>, grid, dim3(128), smem, st, p);
+  else if (vec) sb::launch_pdl(latent_direct_kernel<bf16, true>, grid, dim3(128), smem, st, p);
+  else sb::launch_pdl(latent_direct_kernel<bf16, false>, grid, dim3(128), smem, st, p);
+  return sb::check_launch("sb_op_latent_direct");
+}
+
+// i: 0 in, 1 in_row, 2 in_head, 3 w, 4 out, 5 out_row, 6 out_head, 7 dtype, 8 H, 9 K, 10 N, 11 tail,
+//    12 the gates' first column in a projection's partial sums (flat; 0: no gates), 13 K ranges S, 14 most tokens with a buffer per range, 15 their width
 SB_EXPORT int sb_op_head_linear(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
-  return sb_head_linear(ptr<const void>(op->i[0]), op->i[1], op->i[2], ptr<const void>(op->i[3]), ptr<void>(op->i[4]), op->i[5], op->i[6], (int)op->i[7],
-                        s->n, (int)op->i[8], (int)op->i[9], (int)op->i[10], (int)op->i[11], static_cast<cudaStream_t>(stream));
+  return sb_head_linear_gated(ptr<const void>(op->i[0]), op->i[1], op->i[2], ptr<const void>(op->i[3]), ptr<void>(op->i[4]), op->i[5], op->i[6],
+                              (int)op->i[7], s->n, (int)op->i[8], (int)op->i[9], (int)op->i[10], (int)op->i[11], ptr<const float>(op->i[12]),
+                              partial_count(op->i[13], op->i[14], s->n), static_cast<int64_t>(s->n) * op->i[15], (int)op->i[15],
+                              static_cast<cudaStream_t>(stream));
 }
 
 // i: 0 q, 1 out, 2 dtype, 3 pages, 4 block table, 5 max_pages, 6 page_size, 7 page_stride, 8 v_offset, 9 head_stride, 10 slopes, 11 sinks, 12 H,

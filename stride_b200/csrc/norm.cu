@@ -229,12 +229,12 @@ __global__ void __launch_bounds__(1024) layernorm_kernel(float* __restrict__ h, 
   const float scale = 1.0f / sqrtf(sb::block_sum(sq, red) / static_cast<float>(H) + eps);
   TO* o = out + r * H;
   for (int i = threadIdx.x; i < H; i += blockDim.x)
-    o[i] = sb::narrow<TO>(fmaf((row[i] - mean) * scale, sb::widen(weight[i]), sb::widen(bias[i])));
+    o[i] = sb::narrow<TO>(fmaf((row[i] - mean) * scale, sb::widen(weight[i]), bias != nullptr ? sb::widen(bias[i]) : 0.0f));
 }
 
 }  // namespace
 
-// Layer norm with gain and bias over rows of H; arguments as sb_rmsnorm, plus the bias (of the gain's dtype).
+// Layer norm with gain and bias over rows of H; arguments as sb_rmsnorm, plus the bias (of the gain's dtype; null: none).
 SB_EXPORT int sb_layernorm(float* h, const float* partials, int n_partials, int64_t partial_stride, const void* weight,
                            const void* bias, int weight_dtype, void* out, int out_dtype, int n, int H, float eps, cudaStream_t stream) {
   if (n <= 0) return 0;
@@ -337,7 +337,7 @@ SB_EXPORT int sb_op_rmsnorm(const SbOp* op, const SbStep* s, void* stream) {
                     ptr<void>(op->i[6]), (int)op->i[7], n, (int)op->i[8], static_cast<float>(op->f[0]), static_cast<cudaStream_t>(stream));
 }
 
-// i: as sb_op_rmsnorm, and 10 the bias
+// i: as sb_op_rmsnorm, and 10 the bias (or 0)
 SB_EXPORT int sb_op_layernorm(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   const int n = op->i[9] ? s->wanted : s->n;

@@ -119,7 +119,7 @@ class Engine:
         build_all(sorted(libraries))      # what this model needs, compiled side by side if missing
         # the word into which the tensor-core kernels' bounded waits report; the sampling kernels pass it on to the host
         self._status_device = None
-        if self.device.type == "cuda" and libraries & {"gemm_tc", "attention_tc5", "decode_chain"}:
+        if self.device.type == "cuda" and libraries & {"gemm_tc", "attention_tc5", "decode_chain", "grouped_gemm"}:
             from ..kernels import ops
             self._status_device = ops.shared_status_word(libraries | {"sampling"})
         plan = self.model.tensor_plan()

@@ -50,6 +50,8 @@ SOURCES = {
     "gated_recurrence": "gated_recurrence.cu",
     "rglru": "rglru.cu",
     "delta_rule": "delta_rule.cu",
+    "streams": "streams.cu",
+    "grouped_gemm": "grouped_gemm.cu",
     "runtime": "runtime.cpp",        # host code only: the cache manager's books and the scheduler's decisions
 }
 HOST_FLAGS = ["-O2", "-std=c++17", "-g1", "-shared", "-fPIC", "-fvisibility=hidden"]

@@ -120,6 +120,9 @@ class Linear:
             program.pending = (flat, self.splits, self.out_features)
             return
         program.need_folded("a projection")
+        fresh = program.take_fresh()        # a branch that holds nothing yet: the result is stored, not added
+        if fresh is not None:
+            return self.emit(program, x, fresh)
         if self._tc(x):
             self._tc_op(program, x, program.h, 2)
         else:

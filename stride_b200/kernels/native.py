@@ -137,7 +137,38 @@ class DecodeChain:
         self._lib.sb_chain_reset(self.handle)
 
 
-class StepProgram:
+class _StreamHolder:
+    """The residual stream's buffer as the operations of a program see it."""
+    _h, h_touched, _fresh, _stream = None, False, False, None
+
+    @property
+    def h(self):
+        """The buffer [max_rows, hidden] float32 that operations adding to the stream write into. A block that runs a sublayer on a branch
+        puts the branch's buffer here meanwhile, and learns from `h_touched` whether any operation wrote into it (or only left partial
+        sums pending). Asked for while the branch holds nothing yet (`set_fresh`), it is set to zero first."""
+        self.h_touched = True
+        if self._fresh:
+            self._fresh = False
+            self.add("branch", "sb_op_branch_clear", [self._h, self._h.shape[1]])
+        return self._h if self._h is not None or self._stream is None else self._stream.h
+
+    @h.setter
+    def h(self, buffer):
+        self._h, self.h_touched, self._fresh = buffer, False, False
+
+    def set_fresh(self, buffer) -> None:
+        """Put a branch's buffer in the stream's place whose contents mean nothing: the first projection stores into it."""
+        self.h, self._fresh = buffer, True
+
+    def take_fresh(self):
+        """The branch's buffer if it holds nothing yet (the caller stores into all of it), else None."""
+        if not self._fresh:
+            return None
+        self._fresh, self.h_touched = False, True
+        return self._h
+
+
+class StepProgram(_StreamHolder):
     """The operations of one engine's step, the tile plans its mixers asked for, and what the build of the
     operations shares: the workspace, and which partial sums are pending on the residual stream."""
 
@@ -147,7 +178,6 @@ class StepProgram:
         self.workspace = workspace
         self.max_rows = max_rows
         self.few_tokens = few_tokens          # up to this many tokens a projection leaves one buffer per K range
-        self._h, self.h_touched = None, False # the residual stream [max_rows, hidden] float32 (`h`), and whether it was asked for since it was set
         self.embedding_output = None          # the embedding's rows [max_rows, hidden] float32, when a part reads them again
         self.pending = None                   # (flat buffer, K ranges, width) left by the last projection, or None
         self._libraries: list = []            # per operation: the library its function lives in (for its error text)
@@ -158,22 +188,12 @@ class StepProgram:
         self.chain = None                     # the DecodeChain being built between begin_chain() and end_chain(), if still whole
         self._chain_at = -1                   # the index of the chain's operation
         self.chains: list = []                # finished chains (kept alive; reset after a failed launch)
+        self.streams = None                   # several residual streams side by side, where a model has them (parts/streams.py)
 
     def __del__(self):
         handle, self._handle = getattr(self, "_handle", None), None
         if handle:
             self._lib.sb_program_destroy(handle)
-
-    @property
-    def h(self):
-        """The buffer that operations adding to the stream write into. A block that runs a sublayer on a branch puts the branch's
-        buffer here meanwhile, and learns from `h_touched` whether any operation wrote into it (or only left partial sums pending)."""
-        self.h_touched = True
-        return self._h
-
-    @h.setter
-    def h(self, buffer):
-        self._h, self.h_touched = buffer, False
 
     def __len__(self):
         return self._lib.sb_program_size(self._handle)
@@ -273,7 +293,7 @@ class StepProgram:
             raise RuntimeError(f"operation {k} of the step failed: " + library(self._libraries[k]).sb_last_error().decode(errors="replace"))
 
 
-class ImmediateProgram:
+class ImmediateProgram(_StreamHolder):
     """A step program that launches every operation the moment it is added, on the current torch stream, for the step that a
     `StepContext` describes. A part that has written its share of a step once, as `emit(program, ...)`, gets its `forward(ctx, ...)` from
     it: `with ImmediateProgram(ctx, stream) as program: self.emit(program, ...)`. The operations are the very functions the native
@@ -297,8 +317,16 @@ class ImmediateProgram:
         self.step.static_keys, self.step.max_rows, self.step.n_plans, self.step.ints = ctx.static_keys, R, 0, base
         self.sampled = ctx.sampled if sampled is None else sampled
         self.embedding_output = ctx.embedding_output
-        self._h, self.h_touched, self.pending = None, False, None
+        self.pending = None
         self.chain = None
+
+    @property
+    def streams(self):
+        return self._stream.streams
+
+    @streams.setter
+    def streams(self, state):
+        self._stream.streams = state
 
     def __enter__(self):
         p = self._stream.take_pending() if self._stream is not None else None
@@ -314,15 +342,6 @@ class ImmediateProgram:
             self._stream.set_pending(flat.reshape(-1)[:P * n * M].view(P, n, M))
             self.pending = None
         return False
-
-    @property
-    def h(self):
-        self.h_touched = True
-        return self._h if self._h is not None else self._stream.h
-
-    @h.setter
-    def h(self, buffer):
-        self._h, self.h_touched = buffer, False
 
     def take_pending(self):
         p, self.pending = self.pending, None

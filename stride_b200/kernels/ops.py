@@ -78,10 +78,10 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, slots=No
 
 
 def layernorm(h: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor, partials=None) -> None:
-    """out = (x - mean(x)) / sqrt(var(x) + eps) * weight + bias with x = h (+ partials[0] + partials[1] ...), folded into h
+    """out = (x - mean(x)) / sqrt(var(x) + eps) * weight + bias (None: no bias) with x = h (+ partials[0] + partials[1] ...), folded into h
     in place as `rmsnorm` does."""
     _cuda(h, weight, bias, out, partials)
-    if weight.dtype != bias.dtype:
+    if bias is not None and weight.dtype != bias.dtype:
         raise TypeError("layernorm takes a gain and a bias of one dtype")
     lib, fn = _fn("norm", "sb_layernorm", [c_void_p, c_void_p, c_int, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                            c_int, c_int, c_float, c_void_p])
@@ -174,6 +174,15 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -
     lib, fn = _fn("elementwise", "sb_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     n, I = out.shape
     _check(lib, fn(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), n, I, GATE_ACTIVATIONS[activation], _stream()))
+
+
+def cap_logits(logits: torch.Tensor, scale: float, cap: float) -> None:
+    """logits <- cap tanh(scale logits / cap) in place (cap 0: scale alone), float32."""
+    _cuda(logits)
+    lib, fn = _fn("elementwise", "sb_cap_logits", [c_void_p, c_int64, c_float, c_float, c_void_p])
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise TypeError("cap_logits takes contiguous float32 logits")
+    _check(lib, fn(_ptr(logits), logits.numel(), scale, cap, _stream()))
 
 
 def gather_rows(src: torch.Tensor, rows: torch.Tensor, out: torch.Tensor, partials=None) -> None:
@@ -294,7 +303,7 @@ def gemm_tc_status() -> int:
 
 _status_word = None
 _status_users = {"gemm_tc": "sb_gemm_tc_use_status_word", "attention_tc5": "sb_attention_tc5_use_status_word",
-                 "decode_chain": "sb_decode_chain_use_status_word",
+                 "decode_chain": "sb_decode_chain_use_status_word", "grouped_gemm": "sb_grouped_gemm_use_status_word",
                  "sampling": "sb_sampling_use_status_word"}   # the sampling kernels only read it
 _status_registered: set = set()
 

@@ -1,8 +1,8 @@
 """Interfaces of the parts a model is put together from, and the part registry.
 
 A part knows its own sizes and constants (from its `PartSpec`) and nothing about
-the model it sits in. Seven categories exist: "norm", "position", "mixer",
-"feed_forward", "rewrite", "branch_scale" and "block" (plus "embedding" and "head" at the ends of the model).
+the model it sits in. Eight categories exist: "norm", "position", "mixer",
+"feed_forward", "rewrite", "branch_scale", "streams" and "block" (plus "embedding" and "head" at the ends of the model).
 A new kind is one class registered under a category:
 
     @register_part("mixer", "my_kind")
@@ -29,7 +29,7 @@ from .spec import PartSpec, TensorPlan
 
 _REGISTRY: dict = {}
 
-CATEGORIES = ("norm", "position", "mixer", "feed_forward", "rewrite", "branch_scale", "block", "embedding", "head")
+CATEGORIES = ("norm", "position", "mixer", "feed_forward", "rewrite", "branch_scale", "streams", "block", "embedding", "head")
 
 
 def register_part(category: str, kind: str):
@@ -130,6 +130,11 @@ class Norm(Part):
     def forward(self, ctx, stream, out: torch.Tensor) -> None:
         """out = norm(stream), where `stream` is the ResidualStream (pending partial sums are folded in)."""
         raise NotImplementedError
+
+    def form(self):
+        """(True: a layer norm, False: an RMS norm; gain; bias or None; eps), gain and bias in float32: what a kernel that norms on its way
+        needs. Optional."""
+        raise NotImplementedError(f"{type(self).__name__} has no form for a kernel that norms on its way")
 
 
 class PositionEncoding(Part):

@@ -37,12 +37,16 @@ class Branch(ResidualStream):
         return (self._buffer if self.touched else None), self.take_pending()
 
 
-def emit_on_branch(program, branch: torch.Tensor, emit) -> tuple:
+def emit_on_branch(program, branch: torch.Tensor, emit, fresh: bool = False) -> tuple:
     """Run `emit()` (a part's `emit` that adds to the program's stream) with `branch` in the stream's place; returns (the branch if an
-    operation wrote into it, else None; the partial sums left pending, or None)."""
+    operation wrote into it, else None; the partial sums left pending, or None). `fresh`: the branch's contents mean nothing (whoever takes
+    it in does not set it back to zero); else it is zero."""
     program.need_folded("a sublayer on a branch")
     main = program._h
-    program.h = branch
+    if fresh:
+        program.set_fresh(branch)
+    else:
+        program.h = branch
     try:
         emit()
         return (branch if program.h_touched else None), program.take_pending()
@@ -124,16 +128,25 @@ class BranchRMSNorm(BranchScale):
         emit_fold(program, sources, self.weight, self.size, norm_eps=self.eps)
 
 
+ALWAYS = 1 << 30      # the limit of partial sums that are never added by the kernel that makes them, however many tokens a step has
+
+
+def pending_limit(pending) -> int:
+    """Up to how many tokens partial sums (flat, count, width[, limit of their own]) lie apart; 0: the program's `few_tokens`."""
+    return pending[3] if pending is not None and len(pending) > 3 else 0
+
+
 def emit_fold(program, sources, gain, width: int, norm_eps: float = None) -> None:
     """The operation that takes one or two branches (buffer or None, pending or None, constant) into the program's stream; with
     `norm_eps` their sum is RMS-normed over its row before the gain."""
     if not 1 <= len(sources) <= 2:
         raise ValueError("a fold takes one or two branches")
     (a, pa, ca), (b, pb, cb) = sources[0], sources[1] if len(sources) > 1 else (None, None, 1.0)
-    (fa, Sa, _), (fb, Sb, _) = pa or (None, 1, 0), pb or (None, 1, 0)
+    (fa, Sa), (fb, Sb) = (pa or (None, 1))[:2], (pb or (None, 1))[:2]
     if a is None and fa is None:
         raise ValueError("a branch that nothing wrote into")
-    ints = [program.h, a, fa, Sa, program.few_tokens, b, fb, Sb, gain, gain.dtype if gain is not None else 0, width]
+    ints = [program.h, a, fa, Sa, program.few_tokens, b, fb, Sb, gain, gain.dtype if gain is not None else 0, width,
+            pending_limit(pa), pending_limit(pb)]
     if norm_eps is None:
         program.add("branch", "sb_op_branch_fold", ints, [ca, cb])
     else:       # the branches' sum is RMS-normed over its row on the way

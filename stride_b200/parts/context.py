@@ -68,6 +68,7 @@ class ResidualStream:
     def __init__(self, h: torch.Tensor):
         self.h = h
         self.pending: Optional[torch.Tensor] = None
+        self.streams = None          # several streams side by side, where a model has them (parts/streams.py)
 
     def take_pending(self) -> Optional[torch.Tensor]:
         p, self.pending = self.pending, None

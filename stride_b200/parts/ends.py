@@ -1,7 +1,7 @@
 """The two ends of a decoder: the token embedding and the output head.
 
 Embedding: h = widen(table[token]) (arhaamatiq/stride src/kernels.cu:98-116), times a constant for designs that scale it.
-Head: logits = W x for the rows that want logits; W is `lm_head.weight` if the
+Head: logits = W x for the rows that want logits, times a constant and softly capped, c tanh(logits / c), for designs that do so (32-bit); W is `lm_head.weight` if the
 checkpoint has it, else the embedding table (src/model.cpp:228-232).
 """
 from __future__ import annotations
@@ -48,7 +48,7 @@ class Embedding(Part):
 @register_part("head", "linear")
 class LinearHead(Part):
     """params: vocab_size, hidden_size, tied (True: always the embedding table; False: its own
-    matrix is required; None: its own matrix if the checkpoint has one). tensors: weight, tied_to."""
+    matrix is required; None: its own matrix if the checkpoint has one), scale (1 by default), cap (0: none). tensors: weight, tied_to."""
     graph_safe = True
 
 
@@ -57,6 +57,8 @@ class LinearHead(Part):
         self.vocab = int(spec.params["vocab_size"])
         self.hidden = int(spec.params["hidden_size"])
         self.tied = spec.params.get("tied")
+        self.scale, self.cap = float(spec.params.get("scale", 1.0)), float(spec.params.get("cap") or 0.0)
+        self.plain = self.scale == 1.0 and self.cap == 0.0
         self.linear = None
 
     def tensor_plan(self):
@@ -78,6 +80,10 @@ class LinearHead(Part):
     def forward(self, x, logits):
         """logits[count, vocab] float32 = x . W^T for the normed rows x."""
         self.linear.forward(x, logits)
+        if not self.plain:
+            ops.cap_logits(logits, self.scale, self.cap)
 
     def emit(self, program, x, logits):
         self.linear.emit(program, x, logits, wanted_rows=True)
+        if not self.plain:
+            program.add("elementwise", "sb_op_cap_logits", [logits, self.vocab], [self.scale, self.cap])

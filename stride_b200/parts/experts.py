@@ -13,15 +13,21 @@ csrc/feed_forward.cu; the identity experts' share: csrc/branch.cu.
 
 Two parameters make other routed designs of it. `weights_from` "logits": the stored vector is the router's bias, z = W_r x + b, the
 `top` largest z are chosen and weigh by the softmax over the chosen z alone. `expert` "silu_gated": an expert is
-W_down (silu(W_gate x) * (W_up x)); its gate and up matrices lie one above the other in the side-by-side product."""
+W_down (silu(W_gate x) * (W_up x)); its gate and up matrices lie one above the other in the side-by-side product.
+
+"table_experts": gated experts without a router, chosen by a stored table of token ids; the products run grouped, every expert on the rows
+that chose it (csrc/grouped_gemm.cu)."""
 from __future__ import annotations
 
 import torch
 
 from ..kernels import ops
 from ..kernels.linear import Linear
+from ..kernels.native import ImmediateProgram
 from .base import FeedForward, register_part
-from .spec import TensorPlan
+from .branch import ALWAYS, emit_fold, emit_on_branch
+from .mlp import SwiGLU
+from .spec import PartSpec, TensorPlan
 
 
 @register_part("feed_forward", "polynorm")
@@ -157,3 +163,98 @@ class RoutedFeedForward(FeedForward):
             z = ws.get("routed.z", T, (E * F,), self.env.act_dtype)
             program.add("feed_forward", "sb_op_moe_activate", [up, S, program.few_tokens, weights, X, z, z.dtype, E, F, int(self.gated)])
             self.down.emit_add(program, z, ws.raw("routed.down_partials", (self.down.partial_elems(T),), f32))
+
+
+@register_part("feed_forward", "table_experts")
+class TableExpertsFeedForward(FeedForward):
+    """Gated experts W_down (silu(W_gate x) * (W_up x)) chosen by the token alone: a stored table names `top` experts for every token id, each
+    with weight 1 / top; a shared expert of the same form may run for every token beside them. The step's (token, choice) pairs are sorted
+    by expert and every projection is one launch over the experts in use, each on its own rows (csrc/grouped_gemm.cu); the choices of a
+    token come back as `top` partial sums, which whoever takes the result in adds in their order, beside the shared expert's.
+    params: hidden_size, vocab_size, intermediate_size (of one expert), experts, top, shared (its intermediate size; 0: none).
+    tensors: table [vocab, top], gate, up, down (lists of names, one per expert), shared_gate, shared_up, shared_down."""
+    graph_safe = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        p = spec.params
+        self.hidden, self.vocab, self.intermediate = int(p["hidden_size"]), int(p["vocab_size"]), int(p["intermediate_size"])
+        self.experts, self.top, self.shared_size = int(p["experts"]), int(p["top"]), int(p.get("shared", 0) or 0)
+        if not 0 < self.top <= self.experts or self.experts > 1024:
+            raise ValueError(f"experts by table: {self.top} of {self.experts} experts (at most 1024)")
+        t = spec.tensors
+        self.shared = SwiGLU(PartSpec("gated", {"hidden_size": self.hidden, "intermediate_size": self.shared_size},
+                                      {"gate": t["shared_gate"], "up": t["shared_up"], "down": t["shared_down"]}), env) if self.shared_size else None
+        self.table = self.gate_up = self.down = None
+        self.tensor_core = False
+
+    def tensor_plan(self):
+        t = self.spec.tensors
+        plan = {t["table"]: TensorPlan((self.vocab, self.top), integer=True, below=self.experts)}
+        for name in (*t["gate"], *t["up"]):
+            plan[name] = TensorPlan((self.intermediate, self.hidden))
+        for name in t["down"]:
+            plan[name] = TensorPlan((self.hidden, self.intermediate))
+        if self.shared is not None:
+            plan.update(self.shared.tensor_plan())
+        return plan
+
+    def bind(self, tensors):
+        t = self.spec.tensors
+
+        def one_below_the_other(names):
+            ws = [tensors[n] for n in names]
+            if len({w.dtype for w in ws}) > 1:
+                ws = [w.to(torch.float32) for w in ws]
+            return torch.cat(ws, dim=0).contiguous()
+
+        self.table = tensors[t["table"]].contiguous()
+        low, high = int(self.table.min()), int(self.table.max())
+        if low < 0 or high >= self.experts:
+            raise ValueError(f"experts by table: '{t['table']}' names experts {low} .. {high} of {self.experts}")
+        self.gate_up = one_below_the_other([name for pair in zip(t["gate"], t["up"]) for name in pair])      # [E (F gate rows, F up rows), hidden]
+        self.down = one_below_the_other(t["down"])                                                          # [E hidden, F]
+        self.tensor_core = (self.env.compute_dtype == torch.bfloat16 and self.gate_up.dtype == self.down.dtype == torch.bfloat16
+                            and self.hidden % 8 == 0 and self.intermediate % 8 == 0)
+        if self.shared is not None:
+            self.shared.bind(tensors)
+
+    def weight_bytes(self):
+        """Of a step of one token: its `top` experts and the shared one."""
+        one = (self.gate_up.numel() * self.gate_up.element_size() + self.down.numel() * self.down.element_size()) // self.experts
+        return self.top * one + (self.shared.weight_bytes() if self.shared is not None else 0)
+
+    def kernel_libraries(self):
+        return {"grouped_gemm", "branch"} | (self.shared.kernel_libraries() if self.shared is not None else set())
+
+    def forward(self, ctx, x, stream):
+        with ImmediateProgram(ctx, stream) as program:
+            self.emit(program, x)
+
+    def emit(self, program, x):
+        program.need_folded("experts by table")
+        emit_fold(program, self.emit_sources(program, x), None, self.hidden)
+
+    def emit_sources(self, program, x):
+        """The result as branches with constants, left to the caller to add."""
+        ws, E, top, F, W, tc = program.workspace, self.experts, self.top, self.intermediate, self.hidden, int(self.tensor_core)
+        T, i32, act = ws.max_tokens, torch.int32, self.env.act_dtype
+        order = ws.raw("experts.order", (T * top,), i32)
+        tiles = ws.raw("experts.tiles", (3 * T * top + 1,), i32)
+        lib = "grouped_gemm"
+        program.add(lib, "sb_op_expert_sort", [self.table, self.vocab, top, E, getattr(program, "sampled", None), order, tiles, tc])
+        if tc:
+            xs = ws.raw("experts.x", (T * top, W), act)
+            program.add(lib, "sb_op_expert_gather", [x, x.stride(0), x.element_size(), order, top, xs, W])
+        else:
+            xs = x
+        z = ws.raw("experts.z", (T * top, F), act)
+        program.add(lib, "sb_op_expert_linear", [xs, xs.stride(0), xs.dtype, self.gate_up, self.gate_up.dtype, z, z.dtype, 2 * F, W, E, top, 1,
+                                                 order, tiles, tc])
+        out = ws.raw("experts.out", (T * top * W,), torch.float32)
+        program.add(lib, "sb_op_expert_linear", [z, F, z.dtype, self.down, self.down.dtype, out, out.dtype, W, F, E, top, 0, order, tiles, tc])
+        sources = [(None, (out, top, W, ALWAYS), 1.0 / top)]
+        if self.shared is not None:
+            branch = ws.get("experts.shared", T, (W,), torch.float32)
+            sources.append((*emit_on_branch(program, branch, lambda: self.shared.emit(program, x), fresh=True), 1.0))
+        return sources

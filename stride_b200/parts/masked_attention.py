@@ -11,7 +11,12 @@ j < keep_first (window 0: every earlier key); a learned number per head may join
 [dim unrotated | rot rotated]; W_dkv x = [c' | r]: c = norm(c') is the key/value latent, r, rotated, a key part that all heads share;
 a head's key is [W_uk,h c | r] and its value W_uv,h c. Only [c | r] is cached, one row per token: the key projection is taken into the
 query, q'_h = [W_uk,h^T q_h,unrotated | q_h,rotated], so that q'_h.[c | r] is the head's score, the attention's values are c itself, and
-W_uv,h is applied to the result (per-head products: `head_linear`). Every earlier key is seen; ordinary softmax."""
+W_uv,h is applied to the result (per-head products: `head_linear`). Every earlier key is seen; ordinary softmax.
+
+Parameters make other designs of it: queries may come straight from the input (q_rank 0: q = W_q x, no norm), the rotated part may be
+missing, a sliding window and a learned sink per head work as above, the heads' results may be multiplied element by element by
+sigmoid(W_g x) (`gate`; on the way out of the W_uv products), and a mixer may store no latent of its own (`own_latent` False: no W_dkv): its schedule
+entry then reads the cache of another latent mixer with the same kv_rank, with its own W_uk and W_uv."""
 from __future__ import annotations
 
 import math
@@ -20,6 +25,7 @@ import torch
 
 from ..kernels import ops
 from ..kernels.linear import Linear
+from ..kernels.native import ImmediateProgram
 from .base import CacheNeed, Mixer, part_class, register_part
 from .spec import TensorPlan
 
@@ -156,7 +162,10 @@ class LatentAttentionMixer(Mixer):
     """params: hidden_size, num_heads, key_dim (a head's unrotated query/key elements), rot_dim (its rotated ones), value_dim, q_rank,
     kv_rank, scale, norm_eps, position (a PartSpec of category "position" offering cos_sin for rotary_dim = rot_dim, or None when
     rot_dim is 0). tensors: dq [q_rank, hidden], dq_norm, uq [H (key_dim + rot_dim), q_rank], dkv [kv_rank + rot_dim, hidden], dkv_norm,
-    uk [H key_dim, kv_rank], uv [H value_dim, kv_rank], o [hidden, H value_dim]."""
+    uk [H key_dim, kv_rank], uv [H value_dim, kv_rank], o [hidden, H value_dim].
+    params further: window (0: every earlier key), sink (True: a number per head in the denominator, tensor sink [H]); with q_rank 0 (tensor
+    q [H key_dim, hidden] in place of dq, dq_norm and uq; no rotated part): gate (True: tensor g [H value_dim, hidden]), own_latent (False:
+    the latents are another schedule entry's; no dkv, dkv_norm)."""
     graph_safe = True
 
     def __init__(self, spec, env):
@@ -171,36 +180,59 @@ class LatentAttentionMixer(Mixer):
         self.row = self.kv_rank + self.rot_dim
         if self.row > 640:
             raise ValueError(f"latent attention: a cached row of {self.row} elements exceeds 640, the most the kernel holds")
+        self.window, self.has_sink = int(p.get("window", 0) or 0), bool(p.get("sink"))
+        self.gated, self.own_latent, self.direct = bool(p.get("gate")), bool(p.get("own_latent", True)), self.q_rank == 0
+        if (self.direct and self.rot_dim) or (not self.direct and (self.gated or not self.own_latent)):
+            raise ValueError("latent attention: queries without a latent have no rotated part; gates and another entry's latents go with them")
         pos = p.get("position")
         if (pos is None) != (self.rot_dim == 0):
             raise ValueError("latent attention: a position part goes with rot_dim > 0, and only with it")
         self.position = part_class("position", pos.kind)(pos, env) if pos is not None else None
-        self.down = self.uq = self.o = self.uk = self.uv = self.q_gain = self.kv_gain = None
+        self.down = self.uq = self.o = self.uk = self.uv = self.q_gain = self.kv_gain = self.sinks = None
 
     def tensor_plan(self):
         t, H = self.spec.tensors, self.num_heads
+        if self.direct:
+            plan = {t["q"]: TensorPlan((H * self.key_dim, self.hidden)), t["uk"]: TensorPlan((H * self.key_dim, self.kv_rank)),
+                    t["uv"]: TensorPlan((H * self.value_dim, self.kv_rank)), t["o"]: TensorPlan((self.hidden, H * self.value_dim))}
+            if self.own_latent:
+                plan.update({t["dkv"]: TensorPlan((self.kv_rank, self.hidden)), t["dkv_norm"]: TensorPlan((self.kv_rank,))})
+            if self.gated:
+                plan[t["g"]] = TensorPlan((H * self.value_dim, self.hidden))
+            if self.has_sink:
+                plan[t["sink"]] = TensorPlan((H,), zero_mean=True)
+            return plan
         plan = {t["dq"]: TensorPlan((self.q_rank, self.hidden)), t["dq_norm"]: TensorPlan((self.q_rank,)),
                 t["uq"]: TensorPlan((H * (self.key_dim + self.rot_dim), self.q_rank)),
                 t["dkv"]: TensorPlan((self.kv_rank + self.rot_dim, self.hidden)), t["dkv_norm"]: TensorPlan((self.kv_rank,)),
                 t["uk"]: TensorPlan((H * self.key_dim, self.kv_rank)), t["uv"]: TensorPlan((H * self.value_dim, self.kv_rank)),
                 t["o"]: TensorPlan((self.hidden, H * self.value_dim))}
+        if self.has_sink:
+            plan[t["sink"]] = TensorPlan((H,), zero_mean=True)
         if self.position is not None:
             plan.update(self.position.tensor_plan())
         return plan
 
     def bind(self, tensors):
         t, f32, H = self.spec.tensors, torch.float32, self.num_heads
-        ws = [tensors[t["dq"]], tensors[t["dkv"]]]
-        if ws[0].dtype != ws[1].dtype:
+        if self.direct:          # [queries | key/value latent | gates], those that this mixer has
+            ws = [tensors[t[r]] for r, there in (("q", True), ("dkv", self.own_latent), ("g", self.gated)) if there]
+        else:                    # [q latent | key/value latent | shared rotated key part]
+            ws = [tensors[t["dq"]], tensors[t["dkv"]]]
+            self.uq = Linear(tensors[t["uq"]], self.env.compute_dtype)
+            self.q_gain = tensors[t["dq_norm"]].to(f32).contiguous()
+        if len({w.dtype for w in ws}) > 1:
             ws = [w.to(f32) for w in ws]
-        self.down = Linear(torch.cat(ws, dim=0), self.env.compute_dtype)       # [q latent | key/value latent | shared rotated key part]
-        self.uq = Linear(tensors[t["uq"]], self.env.compute_dtype)
+        self.down = Linear(torch.cat(ws, dim=0), self.env.compute_dtype)
         self.o = Linear(tensors[t["o"]], self.env.compute_dtype)
         act = self.env.act_dtype
         # per head: [key_dim, kv_rank] takes the unrotated query to the latent; [kv_rank, value_dim] takes the latent result to the values
         self.uk = tensors[t["uk"]].to(act).view(H, self.key_dim, self.kv_rank).contiguous()
         self.uv = tensors[t["uv"]].to(act).view(H, self.value_dim, self.kv_rank).transpose(1, 2).contiguous()
-        self.q_gain, self.kv_gain = tensors[t["dq_norm"]].to(f32).contiguous(), tensors[t["dkv_norm"]].to(f32).contiguous()
+        if self.own_latent:
+            self.kv_gain = tensors[t["dkv_norm"]].to(f32).contiguous()
+        if self.has_sink:
+            self.sinks = tensors[t["sink"]].to(f32).contiguous()
         if self.position is None:
             self._cos_sin = torch.zeros(2, device=self.env.device)
         else:
@@ -212,11 +244,11 @@ class LatentAttentionMixer(Mixer):
             self._cos_sin = table
 
     def weight_bytes(self):
-        return (self.down.weight_bytes() + self.uq.weight_bytes() + self.o.weight_bytes()
+        return (self.down.weight_bytes() + (self.uq.weight_bytes() if self.uq is not None else 0) + self.o.weight_bytes()
                 + (self.uk.numel() + self.uv.numel()) * self.uk.element_size())
 
     def cache_need(self):
-        return CacheNeed("pages", kv_heads=1, head_dim=self.row, window=0, dtype=self.env.act_dtype, planes=1)
+        return CacheNeed("pages", kv_heads=1, head_dim=self.row, window=self.window, dtype=self.env.act_dtype, planes=1)
 
     def kernel_libraries(self):
         return {"masked_attention", "gemm_tc" if self.env.compute_dtype == torch.bfloat16 else "gemm_f32"}
@@ -232,6 +264,9 @@ class LatentAttentionMixer(Mixer):
                 ws.get("lattn.out", rows, (H * self.value_dim,), act))
 
     def forward(self, ctx, x, stream, cache):
+        if self.direct:
+            with ImmediateProgram(ctx, stream) as program:
+                return self._emit_direct(program, x, cache)
         n, ws, H, f32 = ctx.n, ctx.workspace, self.num_heads, torch.float32
         Dq, R, rot, V = self.key_dim + self.rot_dim, self.kv_rank, self.rot_dim, self.value_dim
         proj = self.down.forward_partials(x, ws.raw("lattn.proj", (self.down.partial_elems(ws.max_tokens),), f32))
@@ -241,11 +276,35 @@ class LatentAttentionMixer(Mixer):
         qp = self.uq.forward_partials(cq, ws.raw("lattn.q_partials", (self.uq.partial_elems(ws.max_tokens),), f32))
         ops.rotate_heads(qp, ctx.positions, self._cos_sin, q.view(n, H * Dq), H, Dq, self.key_dim, rot)
         ops.head_linear(q, self.uk, ql, tail=rot)
-        _attend(ql.view(n, H * self.row), ol.view(n, H * R), cache, ctx, None, None, H, 1, self.row, R, 0, 0, self.scale, self._tiles(cache.pages))
+        _attend(ql.view(n, H * self.row), ol.view(n, H * R), cache, ctx, None, self.sinks, H, 1, self.row, R, self.window, 0, self.scale,
+                self._tiles(cache.pages))
         ops.head_linear(ol, self.uv, mixed.view(n, H, V))
         self.o.forward_add(mixed, stream, ws.raw("lattn.o_partials", (self.o.partial_elems(ws.max_tokens),), f32))
 
+    def _emit_direct(self, program, x, cache):
+        ws, H, f32, act = program.workspace, self.num_heads, torch.float32, self.env.act_dtype
+        T, few = ws.max_tokens, program.few_tokens
+        D, R, V = self.key_dim, self.kv_rank, self.value_dim
+        if cache.writes != self.own_latent:
+            raise ValueError("latent attention: a mixer that stores latents needs a cache of its own, one that does not another entry's")
+        proj = ws.raw("lattn.direct", (self.down.partial_elems(T),), f32)
+        S = self.down.emit_partials(program, x, proj)
+        width, stored = self.down.out_features, R if self.own_latent else 0
+        q, ql, ol = (ws.get(name, T, tail, act) for name, tail in (("lattn.dq", (H * D,)), ("lattn.ql", (H, R)), ("lattn.ol", (H, R))))
+        mixed = ws.get("lattn.out", T, (H * V,), act)
+        pages, table = cache.pages, cache.block_table
+        program.add("masked_attention", "sb_op_latent_direct",
+                    [proj, width, S, few, self.kv_gain, q, q.dtype, pages, table, table.shape[1], pages.shape[3], pages.stride(0), H * D, stored,
+                     pages.shape[4]], [self.eps])
+        program.add("masked_attention", "sb_op_head_linear", [q, H * D, D, self.uk, ql, H * R, R, q.dtype, H, D, R, 0])
+        _emit_attend(program, ql, ol, cache, None, self.sinks, H, 1, R, R, self.window, 0, self.scale, self._tiles(pages))
+        gate = [proj[H * D + stored:], S, few, width] if self.gated else []
+        program.add("masked_attention", "sb_op_head_linear", [ol, H * R, R, self.uv, mixed, H * V, V, ol.dtype, H, R, V, 0, *gate])
+        self.o.emit_add(program, mixed, ws.raw("lattn.o_partials", (self.o.partial_elems(T),), f32))
+
     def emit(self, program, x, cache):
+        if self.direct:
+            return self._emit_direct(program, x, cache)
         ws, H, f32 = program.workspace, self.num_heads, torch.float32
         T = ws.max_tokens
         Dq, R, rot, V = self.key_dim + self.rot_dim, self.kv_rank, self.rot_dim, self.value_dim
@@ -260,6 +319,6 @@ class LatentAttentionMixer(Mixer):
         S = self.uq.emit_partials(program, cq, qp)
         program.add("masked_attention", "sb_op_rotate_heads", [qp, S, program.few_tokens, self._cos_sin, q, q.dtype, H, Dq, self.key_dim, rot])
         program.add("masked_attention", "sb_op_head_linear", [q, H * Dq, Dq, self.uk, ql, H * self.row, self.row, q.dtype, H, self.key_dim, R, rot])
-        _emit_attend(program, ql, ol, cache, None, None, H, 1, self.row, R, 0, 0, self.scale, self._tiles(pages))
+        _emit_attend(program, ql, ol, cache, None, self.sinks, H, 1, self.row, R, self.window, 0, self.scale, self._tiles(pages))
         program.add("masked_attention", "sb_op_head_linear", [ol, H * R, R, self.uv, mixed, H * V, V, ol.dtype, H, R, V, 0])
         self.o.emit_add(program, mixed, ws.raw("lattn.o_partials", (self.o.partial_elems(T),), f32))

@@ -2,12 +2,16 @@
 schedule gives, final norm and head on the rows whose logits are wanted."""
 from __future__ import annotations
 
+from dataclasses import replace
+
 import torch
 
 from ..kernels import ops
-from .base import BuildEnv, part_class
+from ..kernels.native import ImmediateProgram
+from .base import BuildEnv, CacheNeed, part_class
 from .context import ResidualStream
 from .spec import ModelSpec
+from .streams import emit_read
 
 
 class DecoderModel:
@@ -58,10 +62,24 @@ class DecoderModel:
             p.bind(tensors)
 
     def cache_needs(self) -> list:
-        """Per schedule entry: a CacheNeed, None, or ("shared", j)."""
+        """Per schedule entry: a CacheNeed, None, or ("shared", j). An entry whose pages others read asks for the longest of their windows:
+        a page stays while any of them still sees a token of it."""
         needs = []
-        for e in self.spec.schedule:
-            needs.append(("shared", e.cache_of) if e.cache_of is not None else self.blocks[e.layer].cache_need())
+        for i, e in enumerate(self.spec.schedule):
+            own = self.blocks[e.layer].cache_need()
+            if e.cache_of is None:
+                needs.append(own)
+                continue
+            needs.append(("shared", e.cache_of))
+            lent = needs[e.cache_of]
+            if not isinstance(lent, CacheNeed) or not isinstance(own, CacheNeed) or lent.kind != "pages" or own.kind != "pages":
+                continue
+            form = lambda need: (need.kv_heads, need.head_dim, need.dtype, need.planes)
+            if form(lent) != form(own):
+                raise ValueError(f"schedule entry {i} reads the cache of entry {e.cache_of}, whose rows are {form(lent)}, as {form(own)}")
+            everything = lent.window == 0 or own.window == 0
+            needs[e.cache_of] = replace(lent, window=0 if everything else max(lent.window, own.window),
+                                        keep_first=0 if everything else max(lent.keep_first, own.keep_first))
         return needs
 
     def kernel_libraries(self) -> set:
@@ -94,10 +112,15 @@ class DecoderModel:
             self.blocks[e.layer].forward(ctx, stream, caches[i])
         if count == 0:
             return None        # pending partial sums die with the stream: nobody reads h after the last layer
-        rows = ws.raw("model.head_rows", (ws.max_tokens, H), torch.float32)[:count]
-        ops.gather_rows(stream.h, logit_rows, rows, partials=stream.take_pending())
         x = ws.raw("model.head_x", (ws.max_tokens, H), ctx.act_dtype)[:count]
-        self.final_norm.forward_rows(rows, x)
+        if stream.streams is not None:
+            with ImmediateProgram(ctx, stream) as program:
+                program.step.wanted = count
+                emit_read(program, stream.streams, None, self.final_norm, x, last=True)
+        else:
+            rows = ws.raw("model.head_rows", (ws.max_tokens, H), torch.float32)[:count]
+            ops.gather_rows(stream.h, logit_rows, rows, partials=stream.take_pending())
+            self.final_norm.forward_rows(rows, x)
         if count > self.env.max_logit_rows:
             raise ValueError(f"logits are wanted at {count} places, more than the engine's max_logit_rows {self.env.max_logit_rows}")
         logits = ws.raw("model.logits", (self.env.max_logit_rows, self.spec.vocab_size), torch.float32)[:count]
@@ -125,11 +148,14 @@ class DecoderModel:
             self.blocks[e.layer].emit(program, caches[i])
         if chained:
             program.end_chain()
-        rows = ws.raw("model.head_rows", (ws.max_tokens, H), torch.float32)
-        flat, S, _ = program.take_pending() or (None, 1, 0)
-        program.add("elementwise", "sb_op_gather_rows", [program.h, flat, S, program.few_tokens, rows, H])
         x = ws.raw("model.head_x", (ws.max_tokens, H), self.env.act_dtype)
-        self.final_norm.emit_rows(program, rows, x)
+        if program.streams is not None:      # several streams: their sum on the wanted rows, normed by the same kernel
+            emit_read(program, program.streams, None, self.final_norm, x, last=True)
+        else:
+            rows = ws.raw("model.head_rows", (ws.max_tokens, H), torch.float32)
+            flat, S, _ = program.take_pending() or (None, 1, 0)
+            program.add("elementwise", "sb_op_gather_rows", [program.h, flat, S, program.few_tokens, rows, H])
+            self.final_norm.emit_rows(program, rows, x)
         logits = ws.raw("model.logits", (self.env.max_logit_rows, self.spec.vocab_size), torch.float32)
         self.head.emit(program, x, logits)
         return logits

@@ -22,7 +22,7 @@ class RMSNorm(Norm):
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
         self.offset = float(spec.params.get("offset", 0.0))
-        self.weight = None
+        self.weight = self._form = None
 
     def tensor_plan(self):
         return {self.spec.tensors["weight"]: TensorPlan((self.size,), zero_mean=self.offset != 0.0)}
@@ -34,6 +34,11 @@ class RMSNorm(Norm):
 
     def weight_bytes(self):
         return self.weight.numel() * self.weight.element_size()
+
+    def form(self):
+        if self._form is None:
+            self._form = self.weight.float().contiguous()
+        return False, self._form, None, self.eps
 
     def forward(self, ctx, stream, out):
         ops.rmsnorm(stream.h, self.weight, self.eps, out, partials=stream.take_pending())
@@ -61,28 +66,36 @@ class RMSNorm(Norm):
 @register_part("norm", "layernorm")
 class LayerNorm(Norm):
     """y = (x - mean(x)) / sqrt(var(x) + eps) * w + b, var the mean squared deviation, all in 32-bit.
-    params: size, eps. tensors: weight, bias."""
+    params: size, eps. tensors: weight, and bias for designs that have one."""
     graph_safe = True
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
-        self.weight = self.bias = None
+        self.weight = self.bias = self._form = None
 
     def tensor_plan(self):
         t = self.spec.tensors
-        return {t["weight"]: TensorPlan((self.size,)), t["bias"]: TensorPlan((self.size,), zero_mean=True)}
+        plan = {t["weight"]: TensorPlan((self.size,))}
+        if "bias" in t:
+            plan[t["bias"]] = TensorPlan((self.size,), zero_mean=True)
+        return plan
 
     def bind(self, tensors):
         t = self.spec.tensors
-        w, b = tensors[t["weight"]], tensors[t["bias"]]
-        if w.dtype != b.dtype:
+        w, b = tensors[t["weight"]], tensors[t["bias"]] if "bias" in t else None
+        if b is not None and w.dtype != b.dtype:
             w, b = w.float(), b.float()
-        self.weight, self.bias = w.contiguous(), b.contiguous()
+        self.weight, self.bias = w.contiguous(), b.contiguous() if b is not None else None
 
     def weight_bytes(self):
-        return 2 * self.weight.numel() * self.weight.element_size()
+        return (2 if self.bias is not None else 1) * self.weight.numel() * self.weight.element_size()
+
+    def form(self):
+        if self._form is None:
+            self._form = (self.weight.float().contiguous(), self.bias.float().contiguous() if self.bias is not None else None)
+        return True, *self._form, self.eps
 
     def kernel_libraries(self):
         return {"norm"}

@@ -99,4 +99,6 @@ class TensorPlan:
     shape: tuple
     optional: bool = False
     integer: bool = False
+    below: int = 0               # integers: random ones lie in 0 .. below - 1, those of a row differ
     zero_mean: bool = False      # a vector that is added, not multiplied (a bias): random weights are N(0, .), not 1 + N(0, .)
+    near_identity: bool = False  # a square matrix whose random weights are the identity + N(0, .)

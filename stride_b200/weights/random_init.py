@@ -2,7 +2,8 @@
 configuration and a seed, or the same tensors directly on a device.
 
 Matrices are N(0, std) with std 0.02, norm gains 1 + N(0, gain_std) (0.1 by default, so
-that a norm weight that is dropped or misplaced changes the result), biases N(0, gain_std). Every tensor has its
+that a norm weight that is dropped or misplaced changes the result), biases N(0, gain_std), matrices that mix residual
+streams the identity + N(0, gain_std), rows of integer tables distinct numbers of their range. Every tensor has its
 own generator seeded from (seed, tensor name), so a tensor's values depend on neither
 the order of generation nor the other tensors. arhaamatiq/stride has no such mode in its
 engine; its tests build a tiny model with a Python script (tests/make_tiny_model.py:19-54).
@@ -46,11 +47,18 @@ def random_tensors(config: dict, seed: int, device="cpu", dtype=torch.bfloat16, 
             continue
         gen = torch.Generator(device=device).manual_seed(_tensor_seed(seed, name))
         if want.integer:
-            out[name] = torch.zeros(want.shape, dtype=torch.int32, device=device)
+            if want.below:
+                order = torch.rand((*want.shape[:-1], want.below), generator=gen, device=device).argsort(dim=-1)
+                out[name] = order[..., :want.shape[-1]].to(torch.int32).contiguous()
+            else:
+                out[name] = torch.zeros(want.shape, dtype=torch.int32, device=device)
         elif len(want.shape) == 1 and want.zero_mean:
             out[name] = (gain_std * torch.randn(want.shape, generator=gen, device=device, dtype=torch.float32)).to(dtype)
         elif len(want.shape) == 1:
             out[name] = (1.0 + gain_std * torch.randn(want.shape, generator=gen, device=device, dtype=torch.float32)).to(dtype)
+        elif want.near_identity:
+            noise = gain_std * torch.randn(want.shape, generator=gen, device=device, dtype=torch.float32)
+            out[name] = (torch.eye(want.shape[0], device=device) + noise).to(dtype)
         else:
             out[name] = (std * torch.randn(want.shape, generator=gen, device=device, dtype=torch.float32)).to(dtype)
     return out
