@@ -388,6 +388,17 @@ def _sitivik_config(width: int, ff: int, vocab: int, pairs: int, window: int) ->
             "layers": ([par, dif] * pairs)[:2 * pairs - 1] + [par2]}
 
 
+def _viperax_config(width: int, ff: int, vocab: int, pairs: int, window: int) -> dict:
+    """2 `pairs` layers of windowed latent attention (16 heads of 128 a 2,048 of width, a latent of 512, sink and gate), the last half of
+    them reading the latents of the layer in front; three residual streams; eight experts of ff / 4, one a token, and a shared one of
+    ff / 4 (as many products a token as two of eight)."""
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 8, "top": 1}, "shared": {"ff": ff // 4}}
+    mixer = {"heads": width // 128, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5, "mask": {"size": window}}
+    layers = [{"type": "latent_attention", "mlp": moe, "mixer": mixer if i < pairs else dict(mixer, kv_from=pairs - 1)} for i in range(2 * pairs)]
+    return {"architecture": "Viperax", "vocab": vocab, "width": width, "streams": 3, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_scale": 0.5, "logit_softcap": 15.0, "layers": layers}
+
+
 def design_compare(a) -> int:
     """Keralorn at layer sizes of a real model beside LlamaForCausalLM with as many layers of the same width, heads and
     feed-forward (random weights, bfloat16 engine): a prompt of 2,048 tokens in one step, decode steps at batch 8 and 64
@@ -408,9 +419,13 @@ def design_compare(a) -> int:
         configs = {"pusisun": _pusisun_config(width, ff, vocab, pairs, 1024), "ganupel": _ganupel_config(width, ff, vocab, pairs, 1024), "llama": llama}
     if a.design == "sitivik":      # beside the closest design (windowed attention beside a gated linear attention with a state per request) and Llama
         configs = {"sitivik": _sitivik_config(width, ff, vocab, pairs, 1024), "ganupel": _ganupel_config(width, ff, vocab, pairs, 1024), "llama": llama}
+    if a.design == "viperax":      # beside the closest design (latent attention, routed gated experts of the same sizes), at two widths
+        configs = {"viperax": _viperax_config(width, ff, vocab, pairs, 1024), "pusisun": _pusisun_config(width, ff, vocab, pairs, 1024),
+                   "viperax_width_4096": _viperax_config(4096, 14336, vocab, pairs, 1024),
+                   "pusisun_width_4096": _pusisun_config(4096, 14336, vocab, pairs, 1024)}
     gen = torch.Generator().manual_seed(3)
     out = {"design": a.design, "beside": {"keralorn": "LlamaForCausalLM", "ganupel": "Keralorn, LlamaForCausalLM", "pusisun": "Ganupel, LlamaForCausalLM",
-                                          "sitivik": "Ganupel, LlamaForCausalLM"}[a.design], "width": width, "ff": ff, "layers": layers, "vocab": vocab,
+                                          "sitivik": "Ganupel, LlamaForCausalLM", "viperax": "Pusisun"}[a.design], "width": width, "ff": ff, "layers": layers, "vocab": vocab,
            "dtype": "bf16", "data": "synthetic (random weights and tokens)", "peaks": pk,
            "l2": "weights and caches of a step exceed the 126 MB L2; the kernel timings flush L2 between launches"}
     flush = torch.empty(160 << 20, dtype=torch.uint8, device="cuda")
@@ -488,8 +503,9 @@ def design_compare(a) -> int:
         del eng
         torch.cuda.empty_cache()
 
-    if a.design in ("ganupel", "pusisun", "sitivik"):
-        out["kernels"] = {"ganupel": _ganupel_kernels, "pusisun": _pusisun_kernels, "sitivik": _sitivik_kernels}[a.design](timed, pk, width, ff)
+    if a.design in ("ganupel", "pusisun", "sitivik", "viperax"):
+        out["kernels"] = {"ganupel": _ganupel_kernels, "pusisun": _pusisun_kernels, "sitivik": _sitivik_kernels,
+                          "viperax": _viperax_kernels}[a.design](timed, pk, width, ff)
         out["clocks"] = clocks.stop()
         print(json.dumps(out))
         return 0
@@ -906,6 +922,122 @@ def _sitivik_kernels(timed, pk: dict, width: int, ff: int) -> dict:
     return kern
 
 
+def _viperax_kernels(timed, pk: dict, width: int, ff: int) -> dict:
+    """Viperax's own kernels alone (L2 flushed between launches), each beside the like kernel of Pusisun."""
+    import torch
+    from stride_b200.kernels import ops
+    from stride_b200.kernels.native import ImmediateProgram
+    from stride_b200.parts import Workspace
+    from stride_b200.parts.context import step_context
+    dev, kern, f32, bf, i32 = "cuda", {}, torch.float32, torch.bfloat16, torch.int32
+    hbm = pk["hbm_gbs"] * 1e9
+
+    def record(label, ms, moved=None, flops=None, **more):
+        r = {"ms": round(ms, 4)}
+        if moved is not None:
+            r.update(gb_s=round(moved / ms / 1e6, 1), hbm_fraction_of_measured=round(moved / (ms * 1e-3) / hbm, 3))
+        if flops is not None:
+            r.update(tflops=round(flops / ms / 1e9, 2), fraction_of_measured_bf16=round(flops / ms / 1e9 / pk["bf16_tflops"], 4))
+        r.update(more)
+        kern[label] = r
+
+    ws = Workspace(dev, 2048)
+    H, D, V, R, rot, S, window, page = width // 128, 128, 128, 512, 64, 3, 1024, 64
+    row = R + rot                                    # Pusisun's cached row carries a rotated key part of 64 behind the latent
+    E, F, vocab = 8, ff // 4, 32000
+    rand = lambda *shape: torch.randn(*shape, device=dev)
+    gain = torch.ones(width, device=dev)
+    table = torch.randint(0, E, (vocab, 2), generator=torch.Generator().manual_seed(1)).to(i32).to(dev)
+    table[:, 1] = (table[:, 0] + 1) % E
+    w_up, w_down = (rand(E * 2 * F, width) * 0.02).to(bf), (rand(E * width, F) * 0.02).to(bf)
+    cs = torch.rand(4096, rot // 2, 2, device=dev)
+    for label, entries, length, past in (("prefill_2048", 1, 2048, 0), ("decode_b64", 64, 1, 1500), ("decode_b8", 8, 1, 1500)):
+        n, per = entries * length, (past + length + page - 1) // page
+        toks = torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(2)).tolist()
+        ctx = step_context([(e, length, past) for e in range(entries)], ws, bf, tokens=toks, rows=2048)
+        op = lambda function, ints, floats=(), library="masked_attention": ImmediateProgram(ctx, None).prepared(library, function, ints, floats)
+        block = torch.arange(entries * per, dtype=i32, device=dev).view(entries, per)
+        pages, ppages = rand(entries * per + 1, 1, 1, page, R).to(bf), rand(entries * per + 1, 1, 1, page, row).to(bf)
+        # the attention over the latents: a window and a sink; Pusisun's sees every earlier key
+        ql, ol, sinks = rand(n, H * R).to(bf), torch.empty(n, H * R, dtype=bf, device=dev), torch.zeros(H, device=dev)
+        seen = lambda i: min(window, i + 1)
+        keys = sum(seen(past + t) for t in range(length)) * entries
+        moved = (entries * seen(past) * R * 2.0 + n * H * 2 * R * 2.0) if length == 1 else None
+        ms = timed(op("sb_op_masked_attention_tiles", [ql, ol, pages, block, per, page, pages.stride(0), 0, pages.stride(2), None, sinks, H, 1, R, R, R, window, 0],
+                      [0.09]), 5, clear=True)
+        record("latent_attention_" + label, ms, moved, 4.0 * keys * H * R)
+        pql = rand(n, H * row).to(bf)
+        keys = sum(past + t + 1 for t in range(length)) * entries
+        moved = (entries * (past + 1) * row * 2.0 + n * H * (row + R) * 2.0) if length == 1 else None
+        ms = timed(op("sb_op_masked_attention_tiles", [pql, ol, ppages, block, per, page, ppages.stride(0), 0, ppages.stride(2), None, None, H, 1, row, R, row, 0, 0],
+                      [0.07]), 5, clear=True)
+        record("pusisun_latent_attention_" + label, ms, moved, 2.0 * keys * H * (row + R))
+        # in front of it: queries stored, the latent normed and appended; Pusisun norms two latents and rotates the shared key part
+        wide = H * D + R + H * V
+        proj, q = rand(n * wide), torch.empty(n, H * D, dtype=bf, device=dev)
+        ms = timed(op("sb_op_latent_direct", [proj, wide, 1, 0, gain[:R], q, bf, pages, block, per, page, pages.stride(0), H * D, R, R], [1e-5]), 5, clear=True)
+        record("latent_direct_" + label, ms, n * (H * D + R) * 6.0)
+        pproj, cq = rand(n * (768 + row)), torch.empty(n, 768, dtype=bf, device=dev)
+        ms = timed(op("sb_op_latent_prepare", [pproj, 1, 0, gain[:768], gain[:R], cs, cq, bf, ppages, block, per, page, ppages.stride(0), 768, R, rot, row, 1],
+                      [1e-5]), 5, clear=True)
+        record("pusisun_latent_prepare_" + label, ms, n * (768 + row) * 6.0)
+        # the products per head: the key projection into the queries; the value projection with and without the gate on the way out
+        uk, uv = (rand(H, D, R) * 0.05).to(bf), (rand(H, R, V) * 0.05).to(bf)
+        ms = timed(op("sb_op_head_linear", [q, H * D, D, uk, ql, H * R, R, bf, H, D, R, 0]), 5, clear=True)
+        record("head_linear_keys_into_queries_" + label, ms, n * H * (D + R) * 2.0 + uk.numel() * 2.0, 2.0 * n * H * D * R)
+        mixed = torch.empty(n, H * V, dtype=bf, device=dev)
+        ms = timed(op("sb_op_head_linear", [ol, H * R, R, uv, mixed, H * V, V, bf, H, R, V, 0, proj[H * D + R:], 1, 0, wide]), 5, clear=True)
+        record("head_linear_values_gated_" + label, ms, n * H * (R * 2.0 + V * 6.0) + uv.numel() * 2.0, 2.0 * n * H * R * V)
+        ms = timed(op("sb_op_head_linear", [ol, H * R, R, uv, mixed, H * V, V, bf, H, R, V, 0]), 5, clear=True)
+        record("pusisun_head_linear_values_" + label, ms, n * H * (R + V) * 2.0 + uv.numel() * 2.0, 2.0 * n * H * R * V)
+        # between two sublayers: the streams take a result in and are read, normed; Pusisun: the norm behind a sublayer, and the norm in front
+        P = 1 if n > 512 else 8                      # K ranges of the projection in front, as buffers in steps of few tokens
+        x, parts, br = rand(n * S * width), rand(P, n, width), rand(n, width)
+        mix, coef = torch.eye(S, device=dev), torch.ones(S, device=dev)
+        normed = torch.empty(n, width, dtype=bf, device=dev)
+        ms = timed(op("sb_op_streams_step", [x, S * width, width, x, None, parts, P, 512, None, None, 1, 0, mix, coef, coef, gain, None, 1, normed, bf, S, width, 0],
+                      [1.0, 1.0, 1e-5], "streams"), 5, clear=True)
+        record("streams_step_" + label, ms, n * width * (8.0 * S + 4.0 * P + 2.0))
+        two = rand(1, n, width)
+        ms = timed(op("sb_op_streams_step", [x, S * width, width, x, None, two, 1, 1 << 30, None, parts, P, 512, mix, coef, coef, gain, None, 1, normed, bf, S, width, 0],
+                      [1.0, 1.0, 1e-5], "streams"), 5, clear=True)
+        record("streams_step_two_sources_" + label, ms, n * width * (8.0 * S + 4.0 * P + 6.0))
+        h = rand(n, width)
+        ms = timed(lambda: ops.branch_norm_fold(h, gain, 1e-6, a_partials=parts), 5, clear=True)
+        record("pusisun_branch_norm_fold_" + label, ms, n * width * (8.0 + 4.0 * P))
+        ms = timed(lambda: ops.rmsnorm(h, gain, 1e-6, normed), 5, clear=True)
+        record("pusisun_rmsnorm_" + label, ms, n * width * 6.0)
+        # experts: top 1 and top 2 of eight; Pusisun runs all eight on every row as one product each way
+        for top in (1, 2):
+            tab = table[:, :top].contiguous()
+            order, tiles = torch.empty(n * top, dtype=i32, device=dev), torch.empty(3 * n * top + 1, dtype=i32, device=dev)
+            xe = rand(n, width).to(bf)
+            xs, z, y = (torch.empty(n * top, k, dtype=t, device=dev) for k, t in ((width, bf), (F, bf), (width, f32)))
+            used = len({int(e) for t in toks for e in tab[t].tolist()})
+            note = {"top": top, "experts_in_use": used}
+            lib = "grouped_gemm"
+            ms = timed(op("sb_op_expert_sort", [tab, vocab, top, E, None, order, tiles, 1], (), lib), 5, clear=True)
+            record(f"expert_sort_top{top}_{label}", ms, n * top * 8.0, **note)
+            ms = timed(op("sb_op_expert_gather", [xe, width, 2, order, top, xs, width], (), lib), 5, clear=True)
+            record(f"expert_gather_top{top}_{label}", ms, n * top * width * 4.0, **note)
+            ms = timed(op("sb_op_expert_linear", [xs, width, bf, w_up, bf, z, bf, 2 * F, width, E, top, 1, order, tiles, 1], (), lib), 5, clear=True)
+            record(f"expert_gate_up_top{top}_{label}", ms, used * 2 * F * width * 2.0 + n * top * (width + F) * 2.0, 4.0 * n * top * F * width, **note)
+            ms = timed(op("sb_op_expert_linear", [z, F, bf, w_down, bf, y, f32, width, F, E, top, 0, order, tiles, 1], (), lib), 5, clear=True)
+            record(f"expert_down_top{top}_{label}", ms, used * F * width * 2.0 + n * top * (F * 2.0 + width * 4.0), 2.0 * n * top * F * width, **note)
+        splits = ops.gemm_tc_splits(2 * E * F, width)
+        buf = torch.empty(max(splits if n <= 512 else 1, 1) * n * 2 * E * F, device=dev)
+        ms = timed(op("sb_op_linear_tc", [xe, width, w_up, width, buf, 2 * E * F, width, 1, splits, 0], (), "gemm_tc"), 5, clear=True)
+        record("pusisun_all_experts_gate_up_" + label, ms, E * 2 * F * width * 2.0, 4.0 * n * 2 * F * width, note="products of two of eight experts counted")
+        wd, ze = (rand(width, E * F) * 0.02).to(bf), rand(n, E * F).to(bf)
+        splits = ops.gemm_tc_splits(width, E * F)
+        ms = timed(op("sb_op_linear_tc", [ze, E * F, wd, E * F, buf, width, E * F, 1, splits, 0], (), "gemm_tc"), 5, clear=True)
+        record("pusisun_all_experts_down_" + label, ms, E * F * width * 2.0, 2.0 * n * 2 * F * width, note="products of two of eight experts counted")
+        lg = rand(min(n, 64), vocab)
+        ms = timed(lambda: ops.cap_logits(lg, 0.5, 15.0), 5, clear=True)
+        record("cap_logits_" + label, ms, lg.numel() * 8.0)
+    return kern
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -916,9 +1048,10 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--shape", default="1b", choices=sorted(SHAPES), help="1b: the decode step (default); 3b, 8b: serving runs")
     ap.add_argument("--skip-points", action="store_true", help="skip the batch 1 / 64, float32 and prefill measurements")
-    ap.add_argument("--design", default="", choices=["", "keralorn", "ganupel", "pusisun", "sitivik"],
+    ap.add_argument("--design", default="", choices=["", "keralorn", "ganupel", "pusisun", "sitivik", "viperax"],
                     help="keralorn: prefill and decode of that design beside a Llama of equal layer sizes, and its own kernels alone; "
-                         "ganupel: the same beside Keralorn and Llama; pusisun: the same beside Ganupel and Llama")
+                         "ganupel: the same beside Keralorn and Llama; pusisun: the same beside Ganupel and Llama; "
+                         "viperax: the same beside Pusisun, at two widths")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)

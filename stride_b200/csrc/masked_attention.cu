@@ -510,18 +510,33 @@ __global__ void __launch_bounds__(128) head_linear_tc_kernel(HeadLinearParams p)
     }
     __syncthreads();
   }
+  const bool pairs = (p.gate_width & 1) == 0 && (p.gate_stride & 1) == 0 && (reinterpret_cast<uintptr_t>(p.gate) & 7) == 0;     // (N is even)
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int r = r0 + warp * 16 + (lane >> 2) + half * 8;
     if (r >= p.n) continue;
     bf16* dst = out + static_cast<int64_t>(r) * p.out_row + n0 + (lane & 3) * 2;
+    float2 g[8];
+    if (p.gate != nullptr) {       // the row's eight pairs of gates requested together, their K ranges' sums in ascending order
+      const float* at = p.gate + static_cast<int64_t>(r) * p.gate_width + h * p.N + n0 + (lane & 3) * 2;
+      for (int s = 0; s < p.gate_partials; ++s, at += p.gate_stride) {
+        float2 v[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int c = (i >> 1) * 16 + (i & 1) * 8;
+          v[i] = make_float2(0.0f, 0.0f);
+          if (n0 + c + (lane & 3) * 2 < p.N) v[i] = pairs ? *reinterpret_cast<const float2*>(at + c) : make_float2(at[c], at[c + 1]);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) g[i] = s == 0 ? v[i] : make_float2(g[i].x + v[i].x, g[i].y + v[i].y);
+      }
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const int c = (i >> 1) * 16 + (i & 1) * 8;
-      const int j = n0 + c + (lane & 3) * 2;
-      if (j >= p.N) continue;
+      if (n0 + c + (lane & 3) * 2 >= p.N) continue;
       float a = acc[i][2 * half], b = acc[i][2 * half + 1];
-      if (p.gate != nullptr) a *= head_gate(p, r, h, j), b *= head_gate(p, r, h, j + 1);
+      if (p.gate != nullptr) a *= 1.0f / (1.0f + expf(-g[i].x)), b *= 1.0f / (1.0f + expf(-g[i].y));
       *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(a, b);
     }
   }

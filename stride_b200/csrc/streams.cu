@@ -18,7 +18,7 @@ SB_DEFINE_LAST_ERROR()
 namespace {
 
 using bf16 = __nv_bfloat16;
-constexpr int kInFlight = 8;
+constexpr int kInFlight = 4;
 constexpr int kMaxStreams = 16;
 
 struct Source {
@@ -61,15 +61,16 @@ __device__ __forceinline__ V source_value(const Source& s, int64_t partial_strid
   V v = {};
   if (s.partials != nullptr) {
     const V* p = reinterpret_cast<const V*>(s.partials) + i;
-    V part[kInFlight];
+    v = p[0];
+    for (int k0 = 1; k0 < s.n_partials; k0 += kInFlight) {
+      V part[kInFlight];
 #pragma unroll
-    for (int k = 0; k < kInFlight; ++k)
-      if (k < s.n_partials) part[k] = p[k * partial_stride];
-    v = part[0];
+      for (int k = 0; k < kInFlight; ++k)
+        if (k0 + k < s.n_partials) part[k] = p[(k0 + k) * partial_stride];
 #pragma unroll
-    for (int k = 1; k < kInFlight; ++k)
-      if (k < s.n_partials) v = plus(v, part[k]);
-    for (int k = kInFlight; k < s.n_partials; ++k) v = plus(v, p[k * partial_stride]);
+      for (int k = 0; k < kInFlight; ++k)
+        if (k0 + k < s.n_partials) v = plus(v, part[k]);
+    }
     if (s.buffer != nullptr) v = plus(reinterpret_cast<const V*>(s.buffer)[i], v);
   } else if (s.buffer != nullptr) {
     v = reinterpret_cast<const V*>(s.buffer)[i];
@@ -91,7 +92,7 @@ __device__ __forceinline__ void store(bf16* dst, float4 v) {
 // A block per row; u stays in shared memory between the norm's sums. SM: the most streams (EXACT: their number). V: float4 where the width
 // is a multiple of four and every buffer 16-byte aligned, else float: which one depends on the width and the buffers, never on the rows.
 template <class TO, class V, int SM, bool EXACT>
-__global__ void __launch_bounds__(512) streams_step_kernel(StepParams p) {
+__global__ void __launch_bounds__(256, SM <= 4 ? 3 : 1) streams_step_kernel(StepParams p) {
   extern __shared__ __align__(16) float row_values[];
   __shared__ float red[32];
   __shared__ float coef[kMaxStreams * (kMaxStreams + 2)];       // mix | out | in
@@ -182,7 +183,7 @@ int launch(const StepParams& p, int rows, bool vec, cudaStream_t stream) {
   const size_t smem = static_cast<size_t>(p.W) * sizeof(float);
   vec = vec && p.S <= 4;        // (more streams: one element of each a thread, or the registers do not hold them)
   const int units = vec ? p.W / 4 : p.W;
-  const int threads = units >= 512 ? 512 : units >= 256 ? 256 : 128;
+  const int threads = units >= 256 ? 256 : 128;
 #define SB_STREAMS(V, SM, EXACT)                                                                                                          \
   do {                                                                                                                                    \
     if (smem > 40 * 1024) cudaFuncSetAttribute(streams_step_kernel<TO, V, SM, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
