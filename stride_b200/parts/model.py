@@ -85,7 +85,8 @@ class DecoderModel:
     def kernel_libraries(self) -> set:
         names = {"elementwise", "gemm_tc" if self.env.compute_dtype == torch.bfloat16 else "gemm_f32"}
         for p in self._parts():
-            names |= p.kernel_libraries()
+            if p is not self.final_norm or not all(getattr(b, "norms_itself", False) for b in self.blocks):
+                names |= p.kernel_libraries()
         if self.env.decode_chain and {"gemm_tc", "attention_tc"} <= names:
             names.add("decode_chain")
         return names

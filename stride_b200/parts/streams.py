@@ -103,6 +103,10 @@ class HyperConnection(Part):
 
 class _StreamsBlock(Block):
     graph_safe = True
+    norms_itself = True          # the norms in front of sublayers, and the model's last one, run inside the streams' kernel
+
+    def kernel_libraries(self):
+        return set().union(*(self.parts[role].kernel_libraries() for role, category in self.ROLES.items() if category != "norm"))
 
     def forward(self, ctx, stream, cache):
         with ImmediateProgram(ctx, stream) as program:
