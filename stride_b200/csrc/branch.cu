@@ -11,6 +11,9 @@
 //
 //   y[r, :] = ca * (a + ..)[r, :] + cb * (b + ..)[r, :];   dst[r, j] += gain[j] * y[r, j] / sqrt(mean_j(y[r, j]^2) + eps)
 //
+// A branch may have a factor per row beside its constant (a gate per token), and the new row may be stored a second time as bfloat16, for
+// designs whose next sublayer reads the residual itself.
+//
 // A second kernel adds a row-scaled copy of the sublayer's input: dst[r, :] += (sum of `count` columns of w[r, :]) * x[r, :],
 // what experts that pass their input through contribute to a routed feed-forward. A third adds another stream's rows and one
 // vector to every row: dst[r, :] = ((dst[r, :] + pending sums) + other[r, :]) + vector[:], what stands in front of a pass over a group
@@ -31,7 +34,18 @@ struct Source {
   int n_partials;
   int64_t stride;
   float c;
+  const float* row_factor = nullptr;      // [n]: times c, or null
 };
+__device__ __forceinline__ float factor(const Source& s) {       // (a block is a row)
+  return s.row_factor != nullptr ? __fmul_rn(s.c, s.row_factor[blockIdx.x]) : s.c;
+}
+__device__ __forceinline__ void narrow4(bf16* dst, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 packed;
+  packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+  packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(dst) = packed;
+}
 
 // One element of a branch: its buffer (zero behind the read) plus its partial sums, h + (p0 + p1 + ..).
 template <class V>
@@ -90,11 +104,12 @@ __global__ void __launch_bounds__(256) branch_fold_kernel(float* __restrict__ ds
   sb::grid_dependency_wait();
   const int64_t row = static_cast<int64_t>(blockIdx.x) * W;
   const bool two = b.h != nullptr || b.partials != nullptr;
+  const float ca = factor(a), cb = factor(b);
   if (VEC) {
     for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
       const int64_t i = (row + c) / 4;
-      float4 v = mul(source_value<float4>(a, i), a.c);
-      if (two) v = add(v, mul(source_value<float4>(b, i), b.c));
+      float4 v = mul(source_value<float4>(a, i), ca);
+      if (two) v = add(v, mul(source_value<float4>(b, i), cb));
       if (gain != nullptr) v = mul(v, gain4<TG>(gain, c));
       float4* d = reinterpret_cast<float4*>(dst) + i;
       *d = add(*d, v);
@@ -102,8 +117,8 @@ __global__ void __launch_bounds__(256) branch_fold_kernel(float* __restrict__ ds
   } else {
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
       const int64_t i = row + c;
-      float v = mul(source_value<float>(a, i), a.c);
-      if (two) v = add(v, mul(source_value<float>(b, i), b.c));
+      float v = mul(source_value<float>(a, i), ca);
+      if (two) v = add(v, mul(source_value<float>(b, i), cb));
       if (gain != nullptr) v = mul(v, sb::widen(gain[c]));
       dst[i] = add(dst[i], v);
     }
@@ -116,20 +131,21 @@ __global__ void __launch_bounds__(256) branch_fold_kernel(float* __restrict__ ds
 // buffers alone, never on the rows of the step.
 template <class TG, bool VEC>
 __global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict__ dst, Source a, Source b, const TG* __restrict__ gain, int W,
-                                                               float eps) {
+                                                               float eps, bf16* __restrict__ copy) {
   extern __shared__ __align__(16) float row_values[];
   __shared__ float red[32];
   sb::grid_launch_dependents();
   sb::grid_dependency_wait();
   const int64_t row = static_cast<int64_t>(blockIdx.x) * W;
   const bool two = b.h != nullptr || b.partials != nullptr;
+  const float ca = factor(a), cb = factor(b);
   float sq = 0.0f;
   if (VEC) {
     float4* held = reinterpret_cast<float4*>(row_values);
     for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
       const int64_t i = (row + c) / 4;
-      float4 v = mul(source_value<float4>(a, i), a.c);
-      if (two) v = add(v, mul(source_value<float4>(b, i), b.c));
+      float4 v = mul(source_value<float4>(a, i), ca);
+      if (two) v = add(v, mul(source_value<float4>(b, i), cb));
       held[c / 4] = v;
       sq = fmaf(v.x, v.x, sq), sq = fmaf(v.y, v.y, sq), sq = fmaf(v.z, v.z, sq), sq = fmaf(v.w, v.w, sq);
     }
@@ -138,13 +154,15 @@ __global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict
       float4 v = mul(held[c / 4], scale);
       if (gain != nullptr) v = mul(v, gain4<TG>(gain, c));
       float4* d = reinterpret_cast<float4*>(dst) + (row + c) / 4;
-      *d = add(*d, v);
+      v = add(*d, v);
+      *d = v;
+      if (copy != nullptr) narrow4(copy + row + c, v);
     }
     return;
   }
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
-    float v = mul(source_value<float>(a, row + c), a.c);
-    if (two) v = add(v, mul(source_value<float>(b, row + c), b.c));
+    float v = mul(source_value<float>(a, row + c), ca);
+    if (two) v = add(v, mul(source_value<float>(b, row + c), cb));
     row_values[c] = v;
     sq = fmaf(v, v, sq);
   }
@@ -152,7 +170,9 @@ __global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
     float v = mul(row_values[c], scale);
     if (gain != nullptr) v = mul(v, sb::widen(gain[c]));
-    dst[row + c] = add(dst[row + c], v);
+    v = add(dst[row + c], v);
+    dst[row + c] = v;
+    if (copy != nullptr) copy[row + c] = sb::narrow<bf16>(v);
   }
 }
 
@@ -188,11 +208,11 @@ inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 
 }  // namespace
 
-SB_EXPORT int sb_branch_fold(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, float* b, const float* pb, int nb, int64_t sb_,
-                             float cb, const void* gain, int gain_dtype, int n, int W, cudaStream_t stream) {
+SB_EXPORT int sb_branch_fold_ex(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, const float* ra, float* b, const float* pb, int nb,
+                                int64_t sb_, float cb, const float* rb, const void* gain, int gain_dtype, int n, int W, cudaStream_t stream) {
   if (n <= 0 || W <= 0) return 0;
   if (a == nullptr && pa == nullptr) return sb::fail("sb_branch_fold: the first branch has neither a buffer nor partial sums");
-  const Source A{a, pa, pa ? na : 0, sa, ca}, B{b, pb, pb ? nb : 0, sb_, cb};
+  const Source A{a, pa, pa ? na : 0, sa, ca, ra}, B{b, pb, pb ? nb : 0, sb_, cb, rb};
   const bool vec = W % 4 == 0 && aligned16(dst) && aligned16(a) && aligned16(pa) && aligned16(b) && aligned16(pb) && aligned16(gain) &&
                    sa % 4 == 0 && sb_ % 4 == 0;
   const int threads = W >= 1024 ? 256 : 128;
@@ -210,20 +230,28 @@ SB_EXPORT int sb_branch_fold(float* dst, float* a, const float* pa, int na, int6
   return sb::check_launch("sb_branch_fold");
 }
 
-SB_EXPORT int sb_branch_norm_fold(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, float* b, const float* pb, int nb,
-                                  int64_t sb_, float cb, const void* gain, int gain_dtype, float eps, int n, int W, cudaStream_t stream) {
+SB_EXPORT int sb_branch_fold(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, float* b, const float* pb, int nb, int64_t sb_,
+                             float cb, const void* gain, int gain_dtype, int n, int W, cudaStream_t stream) {
+  return sb_branch_fold_ex(dst, a, pa, na, sa, ca, nullptr, b, pb, nb, sb_, cb, nullptr, gain, gain_dtype, n, W, stream);
+}
+
+// ra, rb [n]: a factor per row on each branch, or null. copy: the new rows as bfloat16, or null.
+SB_EXPORT int sb_branch_norm_fold_ex(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, const float* ra, float* b, const float* pb,
+                                     int nb, int64_t sb_, float cb, const float* rb, const void* gain, int gain_dtype, float eps, void* copy, int n,
+                                     int W, cudaStream_t stream) {
   if (n <= 0 || W <= 0) return 0;
   if (a == nullptr && pa == nullptr) return sb::fail("sb_branch_norm_fold: the first branch has neither a buffer nor partial sums");
-  const Source A{a, pa, pa ? na : 0, sa, ca}, B{b, pb, pb ? nb : 0, sb_, cb};
+  const Source A{a, pa, pa ? na : 0, sa, ca, ra}, B{b, pb, pb ? nb : 0, sb_, cb, rb};
   const size_t smem = static_cast<size_t>(W) * sizeof(float);
   if (smem > 160 * 1024) return sb::fail("sb_branch_norm_fold: a row of %d elements does not fit the row buffer", W);
   const bool vec = W % 4 == 0 && aligned16(dst) && aligned16(a) && aligned16(pa) && aligned16(b) && aligned16(pb) && aligned16(gain) &&
-                   sa % 4 == 0 && sb_ % 4 == 0;
+                   sa % 4 == 0 && sb_ % 4 == 0 && aligned16(copy);
   const int threads = W >= 1024 ? 256 : 128;
 #define SB_NORM_FOLD(TG, VEC)                                                                                                              \
   do {                                                                                                                                     \
     if (smem > 48 * 1024) cudaFuncSetAttribute(branch_norm_fold_kernel<TG, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
-    sb::launch_pdl(branch_norm_fold_kernel<TG, VEC>, dim3(n), dim3(threads), smem, stream, dst, A, B, static_cast<const TG*>(gain), W, eps); \
+    sb::launch_pdl(branch_norm_fold_kernel<TG, VEC>, dim3(n), dim3(threads), smem, stream, dst, A, B, static_cast<const TG*>(gain), W, eps, \
+                   static_cast<bf16*>(copy));                                                                                              \
   } while (0)
   if (gain == nullptr || gain_dtype == 0) {
     if (vec) SB_NORM_FOLD(float, true);
@@ -236,6 +264,11 @@ SB_EXPORT int sb_branch_norm_fold(float* dst, float* a, const float* pa, int na,
   }
 #undef SB_NORM_FOLD
   return sb::check_launch("sb_branch_norm_fold");
+}
+
+SB_EXPORT int sb_branch_norm_fold(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, float* b, const float* pb, int nb,
+                                  int64_t sb_, float cb, const void* gain, int gain_dtype, float eps, int n, int W, cudaStream_t stream) {
+  return sb_branch_norm_fold_ex(dst, a, pa, na, sa, ca, nullptr, b, pb, nb, sb_, cb, nullptr, gain, gain_dtype, eps, nullptr, n, W, stream);
 }
 
 SB_EXPORT int sb_stream_add(float* dst, const float* partials, int n_partials, int64_t stride, const float* other, const void* vector,
@@ -264,28 +297,30 @@ SB_EXPORT int sb_row_scaled_add(float* dst, const void* x, int x_dtype, const fl
 
 // ------------------------------------------------------------------ operations of the native step program (step_ops.h)
 // i: 0 dst, 1 a, 2 a's partial sums (flat), 3 their K ranges S, 4 most tokens with a buffer per range, 5 b, 6 b's partial sums, 7 their S,
-//    8 gain, 9 gain dtype, 10 W, 11 a limit of a's own in place of i[4] (or 0), 12 the same for b
+//    8 gain, 9 gain dtype, 10 W, 11 a limit of a's own in place of i[4] (or 0), 12 the same for b, 13 a factor per row on a (or 0), 14 on b
 // f: 0 ca, 1 cb
 SB_EXPORT int sb_op_branch_fold(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
   const int W = (int)op->i[10];
   const int64_t stride = static_cast<int64_t>(s->n) * W;
-  return sb_branch_fold(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
-                        static_cast<float>(op->f[0]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]), partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n),
-                        stride, static_cast<float>(op->f[1]), ptr<const void>(op->i[8]), (int)op->i[9], s->n, W, static_cast<cudaStream_t>(stream));
+  return sb_branch_fold_ex(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
+                        static_cast<float>(op->f[0]), ptr<const float>(op->i[13]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]),
+                        partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n), stride, static_cast<float>(op->f[1]), ptr<const float>(op->i[14]),
+                        ptr<const void>(op->i[8]), (int)op->i[9], s->n, W, static_cast<cudaStream_t>(stream));
 }
 
-// i: as sb_op_branch_fold      f: 0 ca, 1 cb, 2 eps
+// i: as sb_op_branch_fold, 15 the new rows once more as bfloat16 (or 0)      f: 0 ca, 1 cb, 2 eps
 SB_EXPORT int sb_op_branch_norm_fold(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
   const int W = (int)op->i[10];
   const int64_t stride = static_cast<int64_t>(s->n) * W;
-  return sb_branch_norm_fold(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
-                             static_cast<float>(op->f[0]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]), partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n),
-                             stride, static_cast<float>(op->f[1]), ptr<const void>(op->i[8]), (int)op->i[9], static_cast<float>(op->f[2]), s->n, W,
-                             static_cast<cudaStream_t>(stream));
+  return sb_branch_norm_fold_ex(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
+                             static_cast<float>(op->f[0]), ptr<const float>(op->i[13]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]),
+                             partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n), stride, static_cast<float>(op->f[1]),
+                             ptr<const float>(op->i[14]), ptr<const void>(op->i[8]), (int)op->i[9], static_cast<float>(op->f[2]), ptr<void>(op->i[15]),
+                             s->n, W, static_cast<cudaStream_t>(stream));
 }
 
 // i: 0 dst, 1 pending partial sums (flat, or 0), 2 their K ranges S, 3 most tokens with a buffer per range, 4 the other stream (or 0),

@@ -232,16 +232,22 @@ __global__ void rope_append_vec_kernel(RopeAppendParams p) {
 }
 
 // ------------------------------------------------------------------ swiglu
-// act 0: silu(a) = a / (1 + e^-a); act 1: the tanh form of gelu, 0.5 a (1 + tanh(sqrt(2/pi) (a + 0.044715 a^3)))
+// act 0: silu(a) = a / (1 + e^-a); act 1: the tanh form of gelu, 0.5 a (1 + tanh(sqrt(2/pi) (a + 0.044715 a^3))); act 2: the clamped gate,
+// a sigmoid(slope a) (b + 1) with a capped at `limit` and b kept within +-limit
 template <class TO>
-__global__ void swiglu_kernel(const float* __restrict__ gate_up, TO* __restrict__ out, int n, int I, int act) {
+__global__ void swiglu_kernel(const float* __restrict__ gate_up, TO* __restrict__ out, int n, int I, int act, float limit, float slope) {
   sb::grid_launch_dependents();
   sb::grid_dependency_wait();
   const int64_t total = static_cast<int64_t>(n) * I;
   for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
        i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t r = i / I, c = i % I;
-    const float a = gate_up[r * 2 * I + c], b = gate_up[r * 2 * I + I + c];
+    float a = gate_up[r * 2 * I + c], b = gate_up[r * 2 * I + I + c];
+    if (act == 2) {
+      a = fminf(a, limit), b = fminf(fmaxf(b, -limit), limit);
+      out[i] = sb::narrow<TO>(a / (1.0f + expf(-slope * a)) * (b + 1.0f));
+      continue;
+    }
     const float g = act == 1 ? 0.5f * a * (1.0f + tanhf(0.7978845608028654f * (a + 0.044715f * a * a * a))) : a / (1.0f + expf(-a));
     out[i] = sb::narrow<TO>(g * b);
   }
@@ -359,12 +365,12 @@ SB_EXPORT int sb_rope_append(const float* qkv, int n_partials, int64_t partial_s
   return sb::check_launch("sb_rope_append");
 }
 
-SB_EXPORT int sb_swiglu(const float* gate_up, void* out, int out_dtype, int n, int I, int act, cudaStream_t stream) {
+SB_EXPORT int sb_swiglu_gated(const float* gate_up, void* out, int out_dtype, int n, int I, int act, float limit, float slope, cudaStream_t stream) {
   if (n <= 0) return 0;
   const int64_t total = static_cast<int64_t>(n) * I;
   const int blocks = static_cast<int>((total + 255) / 256 < sb::sm_count() * 16 ? (total + 255) / 256 : sb::sm_count() * 16);
-  if (out_dtype == 0) sb::launch_pdl(swiglu_kernel<float>, blocks, 256, 0, stream, gate_up, static_cast<float*>(out), n, I, act);
-  else if (out_dtype == 1) sb::launch_pdl(swiglu_kernel<bf16>, blocks, 256, 0, stream, gate_up, static_cast<bf16*>(out), n, I, act);
+  if (out_dtype == 0) sb::launch_pdl(swiglu_kernel<float>, blocks, 256, 0, stream, gate_up, static_cast<float*>(out), n, I, act, limit, slope);
+  else if (out_dtype == 1) sb::launch_pdl(swiglu_kernel<bf16>, blocks, 256, 0, stream, gate_up, static_cast<bf16*>(out), n, I, act, limit, slope);
   else return sb::fail("sb_swiglu: unsupported out dtype %d", out_dtype);
   return sb::check_launch("sb_swiglu");
 }
@@ -401,10 +407,16 @@ SB_EXPORT int sb_op_rope_append(const SbOp* op, const SbStep* s, void* stream) {
                         (int)op->i[16], (int)op->i[17], (int)op->i[18], (int)op->i[19], (int)op->i[21], static_cast<cudaStream_t>(stream));
 }
 
-// i: 0 gate_up (float32 [n, 2 I]), 1 out, 2 out dtype, 3 I, 4 the gate's activation (0 silu, 1 tanh form of gelu)
+SB_EXPORT int sb_swiglu(const float* gate_up, void* out, int out_dtype, int n, int I, int act, cudaStream_t stream) {
+  return sb_swiglu_gated(gate_up, out, out_dtype, n, I, act, 0.0f, 0.0f, stream);
+}
+
+// i: 0 gate_up (float32 [n, 2 I]), 1 out, 2 out dtype, 3 I, 4 the gate's activation (0 silu, 1 tanh form of gelu, 2 clamped)
+// f: 0 limit, 1 slope (of the clamped gate)
 SB_EXPORT int sb_op_swiglu(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
-  return sb_swiglu(ptr<const float>(op->i[0]), ptr<void>(op->i[1]), (int)op->i[2], s->n, (int)op->i[3], (int)op->i[4], static_cast<cudaStream_t>(stream));
+  return sb_swiglu_gated(ptr<const float>(op->i[0]), ptr<void>(op->i[1]), (int)op->i[2], s->n, (int)op->i[3], (int)op->i[4], (float)op->f[0], (float)op->f[1],
+                         static_cast<cudaStream_t>(stream));
 }
 
 // The rows whose logits are wanted, with the pending partial sums of the last projection added.

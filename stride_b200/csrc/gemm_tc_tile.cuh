@@ -49,13 +49,26 @@ __device__ __forceinline__ float silu_fast(float g) { return __fdividef(g, 1.0f 
 // The activation of the gate half of a gated feed-forward: 0 = silu, 1 = the tanh form of gelu,
 // 0.5 g (1 + tanh(y)) with y = sqrt(2/pi) (g + 0.044715 g^3), which is g / (1 + e^(-2y)): the same two approximated
 // instructions as silu. The exponent is capped so that the divisor stays where the approximated division is defined.
-enum GateAct { kGateSilu = 0, kGateGeluTanh = 1 };
+// 2 = g sigmoid(slope g) times (u + 1), g capped at `limit` and u kept within +-limit (constants of the gate).
+enum GateAct { kGateSilu = 0, kGateGeluTanh = 1, kGateClamped = 2 };
+struct Gate {
+  int act = kGateSilu;
+  float limit = 0.0f, slope = 0.0f;
+};
 __device__ __forceinline__ float gate_act(float g, int act) {
   if (act == kGateGeluTanh) {
     const float y = 0.7978845608028654f * fmaf(0.044715f * g, g * g, g);
     return __fdividef(g, 1.0f + __expf(fminf(-2.0f * y, 80.0f)));
   }
   return silu_fast(g);
+}
+// What a gated feed-forward keeps of one gate and one up element.
+__device__ __forceinline__ float gated_product(float g, float u, const Gate& gate) {
+  if (gate.act == kGateClamped) {
+    g = fminf(g, gate.limit), u = fminf(fmaxf(u, -gate.limit), gate.limit);
+    return __fdividef(g, 1.0f + __expf(fminf(-gate.slope * g, 80.0f))) * (u + 1.0f);
+  }
+  return gate_act(g, gate.act) * u;
 }
 
 // Rows of one accumulator tile to global memory: out[n, m] = d (kStore) or out[n, m] += d (kAdd). Each thread
@@ -92,9 +105,11 @@ __device__ __forceinline__ void store_tile(uint32_t tmem_row, float* out, int m,
 // The SwiGLU epilogue of one accumulator tile by the four epilogue warps (128 threads that meet on named barrier 1):
 // lanes 0..63 of the tile hold 64 gate rows, lanes 64..127 the matching up rows; out[n, j] = silu(gate) * up as
 // bfloat16, j = tile_m * 64 + row. `quarter` = warp % 4 (the TMEM lanes this warp may read), xch: 16 x 64 floats of
-// shared memory that nothing else uses meanwhile.
+// shared memory that nothing else uses meanwhile. pair_weight (or null): column n stands for pair order[n], whose input is multiplied by
+// pair_weight[order[n]]; both products are linear in it, so the accumulators are.
 __device__ __forceinline__ void swiglu_tile(uint32_t tmem_base, float* xch, bf16* out, int64_t ldo, int tile_m, int half_rows, int n0,
-                                            int N, int BN, int quarter, int lane, bool ok, int act = kGateSilu) {
+                                            int N, int BN, int quarter, int lane, bool ok, const Gate& gate = Gate(),
+                                            const float* pair_weight = nullptr, const int32_t* order = nullptr) {
   const int j = tile_m * 64 + (quarter & 1) * 32 + lane;  // output feature
   for (int c0 = 0; c0 < BN; c0 += 16) {
     float v[16];
@@ -115,8 +130,12 @@ __device__ __forceinline__ void swiglu_tile(uint32_t tmem_base, float* xch, bf16
         const int n = n0 + c0 + cb + c;
         if (n < N) {
           const float other = xch[(cb + c) * 64 + (quarter & 1) * 32 + lane];
-          const float g = quarter >= 2 ? other : v[c], u = quarter >= 2 ? v[8 + c] : other;
-          out[static_cast<int64_t>(n) * ldo + j] = __float2bfloat16_rn(gate_act(g, act) * u);
+          float g = quarter >= 2 ? other : v[c], u = quarter >= 2 ? v[8 + c] : other;
+          if (pair_weight != nullptr) {
+            const float w = pair_weight[order[n]];
+            g *= w, u *= w;
+          }
+          out[static_cast<int64_t>(n) * ldo + j] = __float2bfloat16_rn(gated_product(g, u, gate));
         }
       }
     }

@@ -1,8 +1,10 @@
 // Experts: many small linear layers of which every token uses a few. A step's (token, choice) pairs are sorted by expert, and one launch
 // per projection runs all experts that the step uses, each on its own rows; an expert that nobody chose costs neither products nor bytes.
 //
-// `expert_sort_kernel` (one CTA): the experts of every token come from a stored table of token ids, `top` of them per token; pair
-// p = k n + token stands for the token's k-th choice. It writes the pairs in expert order (which of an expert's pairs comes first does not
+// `expert_choose_kernel`: a warp per token turns a router's logits into the token's `top` experts, those with the largest logits, and their
+// weights, sigmoid(logit) each; one more logit behind the experts' may be turned into a gate per token, its sigmoid.
+// `expert_sort_kernel` (one CTA): the experts of every token come from a stored table of token ids or from the choice above, `top` of them
+// per token; pair p = k n + token stands for the token's k-th choice. It writes the pairs in expert order (which of an expert's pairs comes first does not
 // matter: every row is computed on its own) and the list of row tiles, (expert, first row, end), cut to the tile size of the products.
 // `expert_gather_kernel` copies the tokens' activations into that order, so that a tile's rows lie one behind the other.
 //
@@ -10,7 +12,8 @@
 // rows, K in one range, TMA through a ring of stages) with the tile's expert read from the list; the weights of all experts are one
 // matrix [E M, K]. float32: `grouped_f32_kernel`, the additions of gemm_f32.cu (32 classes of k, joined by a butterfly). Both have two
 // epilogues: the gated product silu(gate) * up of an expert's gate rows and up rows, which stays in expert order, and a store that
-// scatters row p to [k][token], so that the choices of a token are `top` partial sums in a fixed order for whoever adds them.
+// scatters row p to [k][token], so that the choices of a token are `top` partial sums in a fixed order for whoever adds them. Where a pair's
+// weight multiplies the expert's input, it is applied to the two sums in front of the gate, in 32-bit.
 //
 // What a pair's result is depends on its token and expert alone, never on the tile it falls into.
 #include <algorithm>
@@ -32,9 +35,42 @@ constexpr int kThreads = 192;
 constexpr int kSmemBudget = 200 * 1024;
 
 // ------------------------------------------------------------------ routing
+// logits [n][ldz] float32; choice [n][top] the experts by descending logit (the smaller index among equals), weights [top][n] (pair
+// p = k n + token) their sigmoids, gate [n] (or null) the sigmoid of logit E. PER: experts a lane holds.
+__device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+template <int PER>
+__global__ void __launch_bounds__(128) expert_choose_kernel(const float* __restrict__ logits, int ldz, int n, int E, int top,
+                                                            int32_t* __restrict__ choice, float* __restrict__ weights, float* __restrict__ gate) {
+  sb::grid_launch_dependents();
+  sb::grid_dependency_wait();
+  const int row = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  if (row >= n) return;
+  const float* z = logits + static_cast<int64_t>(row) * ldz;
+  float v[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : -INFINITY;
+  if (gate != nullptr && lane == 0) gate[row] = sigmoid(z[E]);
+  uint32_t taken = 0;               // bit i: this lane's i-th expert has been chosen
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int at = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (!((taken >> i) & 1u) && lane + 32 * i < E && (at == 0x7fffffff || v[i] > best)) best = v[i], at = lane + 32 * i;
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+      if (oa != 0x7fffffff && (at == 0x7fffffff || ob > best || (ob == best && oa < at))) best = ob, at = oa;
+    }
+    if ((at & 31) == lane) taken |= 1u << (at >> 5);
+    if (lane == 0) choice[static_cast<int64_t>(row) * top + k] = min(at, E - 1), weights[static_cast<int64_t>(k) * n + row] = sigmoid(best);
+  }
+}
+
 // order [pairs]; tiles: [0] = how many, then (expert, first row, end row) each.
 __global__ void __launch_bounds__(kSortThreads) expert_sort_kernel(const int32_t* __restrict__ tokens, const int32_t* __restrict__ slots,
-                                                                   const int32_t* __restrict__ sampled, const int32_t* __restrict__ table, int vocab,
+                                                                   const int32_t* __restrict__ sampled, const int32_t* __restrict__ table, int vocab,      // vocab 0: the table's rows are the step's tokens
                                                                    int n, int top, int E, int tile, int32_t* __restrict__ order,
                                                                    int32_t* __restrict__ tiles, int max_tiles) {
   __shared__ int count[kMaxExperts], place[kMaxExperts], tile_at[kMaxExperts + 1];
@@ -45,6 +81,7 @@ __global__ void __launch_bounds__(kSortThreads) expert_sort_kernel(const int32_t
   const int pairs = n * top;
   auto expert_of = [&](int p) {
     const int row = p % n;
+    if (vocab == 0) return min(max(table[static_cast<int64_t>(row) * top + p / n], 0), E - 1);
     int tok = tokens[row];
     if (tok == -1 && sampled != nullptr) tok = sampled[slots[row]];
     if (tok < 0 || tok >= vocab) tok = 0;
@@ -98,6 +135,7 @@ struct TcParams {
   int block_n, stages;
   const int32_t* tiles;
   const int32_t* order;
+  const float* pair_weight;      // kSwiglu: a factor on every pair's input, by pair, or null
   int* status;
 };
 
@@ -184,7 +222,8 @@ grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
     tc_fence_after();
     if (EPI == kSwiglu) {
       float* xch = reinterpret_cast<float*>(smem_raw + (smem0 - smem_u32(smem_raw)));      // stage 0 is free by now
-      swiglu_tile(tmem_base, xch, static_cast<bf16*>(p.out), p.half_rows, tile_m, p.half_rows, n0, end, BN, quarter, lane, ok);
+      swiglu_tile(tmem_base, xch, static_cast<bf16*>(p.out), p.half_rows, tile_m, p.half_rows, n0, end, BN, quarter, lane, ok,
+                  Gate(), p.pair_weight, p.order);
     } else {
       const int m = tile_m * kTileM + quarter * 32 + lane;
       for (int c0 = 0; c0 < BN && n0 + c0 < end; c0 += 16) {
@@ -240,7 +279,7 @@ constexpr int kWarps = 4, kF32Rows = 8, kF32Features = 2;
 template <class TX, class TW, class TO, bool VEC, bool GATED>
 __global__ void __launch_bounds__(kWarps * 32) grouped_f32_kernel(const TX* __restrict__ x, int64_t ldx, const TW* __restrict__ w, TO* __restrict__ out,
                                                                   int M, int K, int n, const int32_t* __restrict__ tiles,
-                                                                  const int32_t* __restrict__ order) {
+                                                                  const int32_t* __restrict__ order, const float* __restrict__ pair_weight) {
   sb::grid_launch_dependents();
   sb::grid_dependency_wait();
   if (static_cast<int>(blockIdx.y) >= tiles[0]) return;
@@ -287,8 +326,9 @@ __global__ void __launch_bounds__(kWarps * 32) grouped_f32_kernel(const TX* __re
   for (int j = 0; j < kF32Rows; ++j) {
     if (lane != j || n0 + j >= end) continue;
     if (GATED) {
-      const float g = acc[0][j];
-      out[static_cast<int64_t>(n0 + j) * half + f0] = sb::narrow<TO>((g / (1.0f + expf(-g))) * acc[1][j]);
+      const float weight = pair_weight != nullptr ? pair_weight[order[n0 + j]] : 1.0f;
+      const float g = acc[0][j] * weight, u = acc[1][j] * weight;
+      out[static_cast<int64_t>(n0 + j) * half + f0] = sb::narrow<TO>((g / (1.0f + expf(-g))) * u);
     } else {
 #pragma unroll
       for (int i = 0; i < kF32Features; ++i)
@@ -299,14 +339,14 @@ __global__ void __launch_bounds__(kWarps * 32) grouped_f32_kernel(const TX* __re
 
 template <class TX, class TW, class TO, bool GATED>
 int launch_f32(const void* x, int64_t ldx, const void* w, void* out, int M, int K, int n, int max_tiles, const int32_t* tiles, const int32_t* order,
-               cudaStream_t stream) {
+               const float* pair_weight, cudaStream_t stream) {
   const int features = kWarps * (GATED ? 1 : kF32Features);
   const dim3 grid(((GATED ? M / 2 : M) + features - 1) / features, max_tiles);
   const bool vec = K % 8 == 0 && (ldx * sizeof(TX)) % 16 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
   if (vec) sb::launch_pdl(grouped_f32_kernel<TX, TW, TO, true, GATED>, grid, dim3(kWarps * 32), 0, stream, static_cast<const TX*>(x), ldx,
-                          static_cast<const TW*>(w), static_cast<TO*>(out), M, K, n, tiles, order);
+                          static_cast<const TW*>(w), static_cast<TO*>(out), M, K, n, tiles, order, pair_weight);
   else sb::launch_pdl(grouped_f32_kernel<TX, TW, TO, false, GATED>, grid, dim3(kWarps * 32), 0, stream, static_cast<const TX*>(x), ldx,
-                      static_cast<const TW*>(w), static_cast<TO*>(out), M, K, n, tiles, order);
+                      static_cast<const TW*>(w), static_cast<TO*>(out), M, K, n, tiles, order, pair_weight);
   return sb::check_launch("sb_op_expert_linear");
 }
 
@@ -331,7 +371,25 @@ SB_EXPORT int sb_expert_tile_ints(int tokens, int top, int E) { return 1 + 3 * m
 
 SB_EXPORT void sb_grouped_gemm_use_status_word(int* device_word) { status_word_given() = device_word; }
 
-// i: 0 table [vocab][top], 1 vocab, 2 top, 3 experts, 4 sampled tokens per slot (or 0), 5 order, 6 tiles, 7 products on the tensor cores
+// i: 0 logits, 1 ldz, 2 experts, 3 top, 4 choice [n][top], 5 weights [top][n], 6 gate [n] from the logit behind the experts' (or 0)
+SB_EXPORT int sb_op_expert_choose(const SbOp* op, const SbStep* s, void* stream) {
+  using namespace sbstep;
+  if (s->n <= 0) return SB_OP_SKIPPED;
+  const int ldz = (int)op->i[1], E = (int)op->i[2], top = (int)op->i[3];
+  if (top < 1 || E < top || E > kMaxExperts || ldz < E + (op->i[6] != 0 ? 1 : 0))
+    return sb::fail("sb_op_expert_choose: %d of %d experts (at most %d) in rows of %d logits", top, E, kMaxExperts, ldz), SB_OP_FAILED;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+#define SB_CHOOSE(PER)                                                                                                                   \
+  sb::launch_pdl(expert_choose_kernel<PER>, dim3((s->n + 3) / 4), dim3(128), 0, st, ptr<const float>(op->i[0]), ldz, s->n, E, top,       \
+                 ptr<int32_t>(op->i[4]), ptr<float>(op->i[5]), ptr<float>(op->i[6]))
+  if (E <= 32) SB_CHOOSE(1);
+  else if (E <= 128) SB_CHOOSE(4);
+  else SB_CHOOSE(32);
+#undef SB_CHOOSE
+  return sb::check_launch("sb_op_expert_choose");
+}
+
+// i: 0 table [vocab][top], 1 vocab (0: the table is the step's choice [n][top]), 2 top, 3 experts, 4 sampled tokens per slot (or 0), 5 order, 6 tiles, 7 products on the tensor cores
 SB_EXPORT int sb_op_expert_sort(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
@@ -363,7 +421,8 @@ SB_EXPORT int sb_op_expert_gather(const SbOp* op, const SbStep* s, void* stream)
 }
 
 // i: 0 x (tensor cores: rows in expert order; 32-bit gated: rows by token), 1 ldx, 2 x dtype, 3 weights [E M][K], 4 their dtype, 5 out, 6 out dtype,
-//    7 M, 8 K, 9 experts, 10 top, 11 gated (1) or scattered store (0), 12 order, 13 tiles, 14 on the tensor cores
+//    7 M, 8 K, 9 experts, 10 top, 11 gated (1) or scattered store (0), 12 order, 13 tiles, 14 on the tensor cores,
+//    15 a factor on every pair's input [top][n] float32 (gated only; 0: none)
 SB_EXPORT int sb_op_expert_linear(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
@@ -374,7 +433,9 @@ SB_EXPORT int sb_op_expert_linear(const SbOp* op, const SbStep* s, void* stream)
   const void* x = ptr<const void>(op->i[0]);
   const void* w = ptr<const void>(op->i[3]);
   void* out = ptr<void>(op->i[5]);
+  const float* pair_weight = ptr<const float>(op->i[15]);
   const int64_t ldx = op->i[1];
+  if (pair_weight != nullptr && !gated) return sb::fail("sb_op_expert_linear: factors on the pairs' inputs go with the gated product"), SB_OP_FAILED;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (M <= 0 || K <= 0 || (gated && M % 2 != 0)) return sb::fail("sb_op_expert_linear: %d x %d", M, K), SB_OP_FAILED;
   const int tile = tile_rows(pairs, E, tc), max_tiles = most_tiles(pairs, E, tile);
@@ -382,8 +443,8 @@ SB_EXPORT int sb_op_expert_linear(const SbOp* op, const SbStep* s, void* stream)
   if (!tc) {
     const int xd = (int)op->i[2], wd = (int)op->i[4], od = (int)op->i[6];
 #define SB_EXPERT(TX, TW, TO)                                                                                              \
-  (gated ? launch_f32<TX, TW, TO, true>(x, ldx, w, out, M, K, s->n, max_tiles, tiles, order, st)                            \
-         : launch_f32<TX, TW, float, false>(x, ldx, w, out, M, K, s->n, max_tiles, tiles, order, st))
+  (gated ? launch_f32<TX, TW, TO, true>(x, ldx, w, out, M, K, s->n, max_tiles, tiles, order, pair_weight, st)               \
+         : launch_f32<TX, TW, float, false>(x, ldx, w, out, M, K, s->n, max_tiles, tiles, order, pair_weight, st))
     if (xd == 0 && wd == 0) return SB_EXPERT(float, float, float);
     if (xd == 0 && wd == 1) return SB_EXPERT(float, bf16, float);
     if (xd == 1 && wd == 0) return SB_EXPERT(bf16, float, bf16);
@@ -394,7 +455,7 @@ SB_EXPORT int sb_op_expert_linear(const SbOp* op, const SbStep* s, void* stream)
   if (K % 8 != 0 || ldx % 8 != 0 || ((op->i[0] | op->i[3]) & 15) != 0)
     return sb::fail("sb_op_expert_linear: K %d and the leading dimension %lld must be multiples of 8, operands 16-byte aligned", K, (long long)ldx), SB_OP_FAILED;
   TcParams p{};
-  p.out = out, p.M = M, p.K = K, p.half_rows = M / 2, p.tiles = tiles, p.order = order, p.block_n = tile;
+  p.out = out, p.M = M, p.K = K, p.half_rows = M / 2, p.tiles = tiles, p.order = order, p.block_n = tile, p.pair_weight = pair_weight;
   p.status = status_word();
   if (!p.status) return sb::fail("sb_op_expert_linear: cannot allocate the status word"), SB_OP_FAILED;
   const int stage_bytes = kStageA + tile * 128;

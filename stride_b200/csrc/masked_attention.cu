@@ -1,6 +1,7 @@
 // Softmax attention over the paged cache with the masks and score terms that grouped-query and latent attention designs combine:
 //
-//   score(i, j) = scale * (q_i . k_j) - slope_h * (i - j)                 slope_h = 0: no distance term
+//   score(i, j) = cap(scale * (q_i . k_j)) - slope_h * (i - j)            slope_h = 0: no distance term
+//   cap(s)      = c tanh(s / c) for designs that cap their scores, else s
 //   i sees j    if j <= i and (window = 0 or i - j < window or j < keep_first) and (chunk = 0 or floor(i / chunk) = floor(j / chunk))
 //   o_i         = sum_j exp(score(i, j) - m) v_j / (sum_j exp(score(i, j) - m) + exp(sink_h - m))      without a sink: no second term
 //
@@ -345,6 +346,7 @@ struct AttnParams {
   float scale;
   int chunk;                 // > 0: a row sees only the keys of its own chunk of this many positions (borders at multiples of it)
   int out_f32;               // 1: `out` is float32 whatever the storage of q and the cache
+  float cap;                 // > 0: scores are capped softly
 };
 
 constexpr int kWarps = 4;
@@ -387,7 +389,9 @@ __global__ void __launch_bounds__(kWarps * 32) masked_attention_kernel(AttnParam
       vr[i] = lane + 32 * i < p.Dv ? sb::widen(v[lane + 32 * i]) : 0.0f;
     }
     for (int o = 16; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-    const float s = __fsub_rn(__fmul_rn(dot, p.scale), __fmul_rn(slope, static_cast<float>(pos - j)));
+    float s = __fmul_rn(dot, p.scale);
+    if (p.cap > 0.0f) s = __fmul_rn(p.cap, tanhf(s / p.cap));
+    s = __fsub_rn(s, __fmul_rn(slope, static_cast<float>(pos - j)));
     const float m_new = fmaxf(m, s);
     const float f = expf(m - m_new), w = expf(s - m_new);       // (m = -inf at the first key: f = 0)
     l = fmaf(l, f, w);
@@ -559,7 +563,14 @@ struct TileParams {
   int stages;                // 2: the next tile of keys is fetched while this one is worked on; 1: after it (half the shared memory)
   int chunk;                 // > 0: a row sees only the keys of its own chunk of this many positions
   int out_f32;               // 1: `out` is float32
+  float cap;                 // > 0: scores are capped softly
 };
+
+// c tanh(s / c) = c - 2 c / (1 + e^(2 s / c)): within a few units of 2^-23 c, with the hardware's approximations of e^x and of the division.
+// (The exponent is capped so that the divisor stays where the approximated division is defined.)
+__device__ __forceinline__ float soft_cap(float s, float c, float two_over_c) {
+  return fmaf(-2.0f * c, __fdividef(1.0f, 1.0f + __expf(fminf(__fmul_rn(s, two_over_c), 80.0f))), c);
+}
 
 constexpr int KT = 64, NK = KT / 16;
 
@@ -606,6 +617,7 @@ __global__ void __launch_bounds__(128) masked_attention_tile_kernel(TileParams p
     if (t < nt) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<int64_t>(row0 + t0 + t) * p.H + head0 + r % Ht) * p.D + c * 8);
     *reinterpret_cast<uint4*>(Qs + r * ldk + c * 8) = v;
   }
+  const float two_over_cap = p.cap > 0.0f ? 2.0f / p.cap : 0.0f;
   const int r_lo = lane >> 2, r_hi = r_lo + 8;
   const int p_lo = r_lo / Ht < nt ? first_pos + r_lo / Ht : -1, p_hi = r_hi / Ht < nt ? first_pos + r_hi / Ht : -1;
   const int h_lo = head0 + r_lo % Ht, h_hi = head0 + r_hi % Ht;
@@ -708,13 +720,23 @@ __global__ void __launch_bounds__(128) masked_attention_tile_kernel(TileParams p
       for (int e = 0; e < 4; ++e) s[i][e] = CH == 4 ? (s4[0][i][e] + s4[CH > 1 ? 1 : 0][i][e]) + (s4[CH > 2 ? 2 : 0][i][e] + s4[CH > 3 ? 3 : 0][i][e]) : s4[0][i][e];
     float top_lo = -INFINITY, top_hi = -INFINITY;
 #pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[i][e] = __fmul_rn(s[i][e], p.scale);
+    if (p.cap > 0.0f) {
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[i][e] = soft_cap(s[i][e], p.cap, two_over_cap);
+    }
+#pragma unroll
     for (int n = 0; n < 2; ++n) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int j = kt * KT + warp * 16 + n * 8 + (lane & 3) * 2 + (c & 1);
         const int pos = c < 2 ? p_lo : p_hi;
         const bool seen = j <= pos && (p.window <= 0 || pos - j < p.window || j < p.keep_first) && (p.chunk <= 0 || j >= pos / p.chunk * p.chunk);
-        const float x = seen ? __fsub_rn(__fmul_rn(s[n][c], p.scale), __fmul_rn(c < 2 ? s_lo : s_hi, static_cast<float>(pos - j))) : -INFINITY;
+        const float x = seen ? __fsub_rn(s[n][c], __fmul_rn(c < 2 ? s_lo : s_hi, static_cast<float>(pos - j))) : -INFINITY;
         s[n][c] = x;
         if (c < 2) top_lo = fmaxf(top_lo, x);
         else top_hi = fmaxf(top_hi, x);
@@ -949,14 +971,14 @@ SB_EXPORT int sb_head_linear(const void* in, int64_t in_row, int64_t in_head, co
 SB_EXPORT int sb_masked_attention_ex(const void* q, void* out, int dtype, const void* pages, const int32_t* block_table, int max_pages, int page_size,
                                      int64_t page_stride, int64_t v_offset, int64_t head_stride, const int32_t* positions, const int32_t* slots,
                                      const float* slopes, const float* sinks, int n, int H, int G, int D, int Dv, int Dc, int window, int keep_first,
-                                     float scale, int chunk, int out_f32, cudaStream_t stream) {
+                                     float scale, int chunk, int out_f32, float cap, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (chunk < 0) return sb::fail("sb_masked_attention: chunk %d", chunk);
   if (H <= 0 || G <= 0 || H % G != 0) return sb::fail("sb_masked_attention: %d heads do not divide into %d key/value heads", H, G);
   if (D <= 0 || Dv <= 0 || D > 640 || Dv > 640) return sb::fail("sb_masked_attention: key size %d, value size %d (at most 640)", D, Dv);
   if (window < 0 || keep_first < 0) return sb::fail("sb_masked_attention: window %d, kept first tokens %d", window, keep_first);
   AttnParams p{q, out, pages, block_table, max_pages, page_size, page_stride, v_offset, head_stride, positions, slots, slopes, sinks,
-               H, G, D, Dv, Dc, window, keep_first, scale, chunk, out_f32};
+               H, G, D, Dv, Dc, window, keep_first, scale, chunk, out_f32, cap};
   const size_t smem = sizeof(float) * (D + kWarps * Dv + 2 * kWarps);
   const bool small = D <= 256 && Dv <= 256;
   if (dtype == 0) {
@@ -976,7 +998,7 @@ SB_EXPORT int sb_masked_attention(const void* q, void* out, int dtype, const voi
                                   const float* slopes, const float* sinks, int n, int H, int G, int D, int Dv, int Dc, int window, int keep_first,
                                   float scale, cudaStream_t stream) {
   return sb_masked_attention_ex(q, out, dtype, pages, block_table, max_pages, page_size, page_stride, v_offset, head_stride, positions, slots, slopes,
-                                sinks, n, H, G, D, Dv, Dc, window, keep_first, scale, 0, 0, stream);
+                                sinks, n, H, G, D, Dv, Dc, window, keep_first, scale, 0, 0, 0.0f, stream);
 }
 
 // The tensor-core form: whether it takes a shape, and the launch. Entries come from the step's records on the device (meta).
@@ -991,14 +1013,14 @@ SB_EXPORT int sb_masked_attention_tiles_supported(int H, int G, int D, int Dv, i
 SB_EXPORT int sb_masked_attention_tiles_ex(const void* q, void* out, const void* pages, const int32_t* block_table, int max_pages, int page_size,
                                            int64_t page_stride, int64_t v_offset, int64_t head_stride, const int32_t* meta, int meta_stride,
                                            int entries, const float* slopes, const float* sinks, int n, int H, int G, int D, int Dv, int Dc,
-                                           int window, int keep_first, float scale, int chunk, int out_f32, cudaStream_t stream) {
+                                           int window, int keep_first, float scale, int chunk, int out_f32, float cap, cudaStream_t stream) {
   if (n <= 0 || entries <= 0) return 0;
   if (chunk < 0) return sb::fail("sb_masked_attention_tiles: chunk %d", chunk);
   if (!sb_masked_attention_tiles_supported(H, G, D, Dv, Dc, v_offset))
     return sb::fail("sb_masked_attention_tiles: heads %d / %d, key size %d, value size %d are not a shape of the tensor-core form", H, G, D, Dv);
   if (window < 0 || keep_first < 0) return sb::fail("sb_masked_attention_tiles: window %d, kept first tokens %d", window, keep_first);
   TileParams p{static_cast<const bf16*>(q), static_cast<bf16*>(out), static_cast<const bf16*>(pages), block_table, max_pages, page_size, page_stride,
-               v_offset, head_stride, meta, meta_stride, entries, slopes, sinks, H, G, D, Dv, Dc, window, keep_first, scale, 2, chunk, out_f32};
+               v_offset, head_stride, meta, meta_stride, entries, slopes, sinks, H, G, D, Dv, Dc, window, keep_first, scale, 2, chunk, out_f32, cap};
   const int groups = (Dv / 16 + 3) / 4;
   switch (groups) {
     case 1: return launch_tiles<1>(p, n, stream);
@@ -1013,7 +1035,7 @@ SB_EXPORT int sb_masked_attention_tiles(const void* q, void* out, const void* pa
                                         const float* slopes, const float* sinks, int n, int H, int G, int D, int Dv, int Dc, int window, int keep_first,
                                         float scale, cudaStream_t stream) {
   return sb_masked_attention_tiles_ex(q, out, pages, block_table, max_pages, page_size, page_stride, v_offset, head_stride, meta, meta_stride, entries,
-                                      slopes, sinks, n, H, G, D, Dv, Dc, window, keep_first, scale, 0, 0, stream);
+                                      slopes, sinks, n, H, G, D, Dv, Dc, window, keep_first, scale, 0, 0, 0.0f, stream);
 }
 
 // ------------------------------------------------------------------ operations of the native step program (step_ops.h)
@@ -1091,25 +1113,27 @@ SB_EXPORT int sb_op_head_linear(const SbOp* op, const SbStep* s, void* stream) {
 }
 
 // i: 0 q, 1 out, 2 dtype, 3 pages, 4 block table, 5 max_pages, 6 page_size, 7 page_stride, 8 v_offset, 9 head_stride, 10 slopes, 11 sinks, 12 H,
-//    13 G, 14 D, 15 Dv, 16 Dc, 17 window, 18 keep_first, 19 chunk, 20 the result as float32      f: 0 scale
+//    13 G, 14 D, 15 Dv, 16 Dc, 17 window, 18 keep_first, 19 chunk, 20 the result as float32      f: 0 scale, 1 soft cap of the scores (0: none)
 SB_EXPORT int sb_op_masked_attention(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
   return sb_masked_attention_ex(ptr<const void>(op->i[0]), ptr<void>(op->i[1]), (int)op->i[2], ptr<const void>(op->i[3]), ptr<const int32_t>(op->i[4]),
                              (int)op->i[5], (int)op->i[6], op->i[7], op->i[8], op->i[9], positions(s), slots(s), ptr<const float>(op->i[10]),
                              ptr<const float>(op->i[11]), s->n, (int)op->i[12], (int)op->i[13], (int)op->i[14], (int)op->i[15], (int)op->i[16],
-                             (int)op->i[17], (int)op->i[18], (float)op->f[0], (int)op->i[19], (int)op->i[20], static_cast<cudaStream_t>(stream));
+                             (int)op->i[17], (int)op->i[18], (float)op->f[0], (int)op->i[19], (int)op->i[20], (float)op->f[1],
+                             static_cast<cudaStream_t>(stream));
 }
 
 // i: 0 q, 1 out, 2 pages, 3 block table, 4 max_pages, 5 page_size, 6 page_stride, 7 v_offset, 8 head_stride, 9 slopes, 10 sinks, 11 H, 12 G, 13 D,
-//    14 Dv, 15 Dc, 16 window, 17 keep_first, 18 chunk, 19 the result as float32      f: 0 scale
+//    14 Dv, 15 Dc, 16 window, 17 keep_first, 18 chunk, 19 the result as float32      f: 0 scale, 1 soft cap of the scores (0: none)
 SB_EXPORT int sb_op_masked_attention_tiles(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   if (s->n <= 0) return SB_OP_SKIPPED;
   return sb_masked_attention_tiles_ex(ptr<const void>(op->i[0]), ptr<void>(op->i[1]), ptr<const void>(op->i[2]), ptr<const int32_t>(op->i[3]), (int)op->i[4],
                                    (int)op->i[5], op->i[6], op->i[7], op->i[8], entry_meta(s), s->max_rows, s->entries, ptr<const float>(op->i[9]),
                                    ptr<const float>(op->i[10]), s->n, (int)op->i[11], (int)op->i[12], (int)op->i[13], (int)op->i[14], (int)op->i[15],
-                                   (int)op->i[16], (int)op->i[17], (float)op->f[0], (int)op->i[18], (int)op->i[19], static_cast<cudaStream_t>(stream));
+                                   (int)op->i[16], (int)op->i[17], (float)op->f[0], (int)op->i[18], (int)op->i[19], (float)op->f[1],
+                                   static_cast<cudaStream_t>(stream));
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------------

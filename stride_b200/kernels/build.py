@@ -52,6 +52,7 @@ SOURCES = {
     "delta_rule": "delta_rule.cu",
     "streams": "streams.cu",
     "grouped_gemm": "grouped_gemm.cu",
+    "short_conv": "short_conv.cu",
     "runtime": "runtime.cpp",        # host code only: the cache manager's books and the scheduler's decisions
 }
 HOST_FLAGS = ["-O2", "-std=c++17", "-g1", "-shared", "-fPIC", "-fvisibility=hidden"]

@@ -88,13 +88,13 @@ class Linear:
         program.add("gemm_f32", "sb_op_linear_f32", [x, x.dtype, x.stride(0), self.weight, self.weight.dtype, self.weight.stride(0), out, ldo,
                                                       self.out_features, self.in_features, int(accumulate), int(wanted_rows)])
 
-    def _tc_op(self, program, x, out, mode: int, splits: int = 1, wanted_rows: bool = False) -> None:
+    def _tc_op(self, program, x, out, mode: int, splits: int = 1, wanted_rows: bool = False, constants=()) -> None:
         # the decode chain has phases for partial sums per K range and for SwiGLU, on the step's tokens
         phase = None
-        if not wanted_rows and mode in (1, 3):      # (the chain's gated epilogue is silu's: mode 4 has no phase)
+        if not wanted_rows and mode in (1, 3):      # (the chain's gated epilogue is silu's: modes 4 and 5 have no phase)
             phase = lambda chain: chain.linear(x, self.weight, out, mode == 3, splits if mode == 1 else 1)
         program.add("gemm_tc", "sb_op_linear_tc", [x, x.stride(0), self.weight, self.weight.stride(0), out, self.out_features,
-                                                    self.in_features, mode, splits, int(wanted_rows)], chain=phase)
+                                                    self.in_features, mode, splits, int(wanted_rows)], constants, chain=phase)
 
     def emit(self, program, x: torch.Tensor, out: torch.Tensor, wanted_rows: bool = False) -> None:
         """`forward`; with `wanted_rows` the rows are the step's wanted rows (the head), not its tokens."""
@@ -128,23 +128,24 @@ class Linear:
         else:
             self._f32_op(program, x, program.h, program.h.stride(0), True, False)
 
-    def emit_swiglu(self, program, x: torch.Tensor, z: torch.Tensor, scratch_fn, activation: str = "silu") -> None:
+    def emit_swiglu(self, program, x: torch.Tensor, z: torch.Tensor, scratch_fn, activation: str = "silu", constants=()) -> None:
         """`forward_swiglu`."""
         act = ops.GATE_ACTIVATIONS[activation]
         if self._tc(x) and z.dtype == torch.bfloat16:
-            self._tc_op(program, x, z, 3 + act)
+            self._tc_op(program, x, z, 3 + act, constants=constants)
         else:
             gate_up = scratch_fn()
             self._f32_op(program, x, gate_up, gate_up.stride(0), False, False)
-            program.add("elementwise", "sb_op_swiglu", [gate_up, z, z.dtype, self.out_features // 2, act])
+            program.add("elementwise", "sb_op_swiglu", [gate_up, z, z.dtype, self.out_features // 2, act], constants)
 
-    def forward_swiglu(self, x: torch.Tensor, z: torch.Tensor, scratch_fn, activation: str = "silu") -> None:
-        """W = [gate rows; up rows]: z[n, I] = act(x . gate^T) * (x . up^T), act = silu or the tanh form of gelu.
+    def forward_swiglu(self, x: torch.Tensor, z: torch.Tensor, scratch_fn, activation: str = "silu", constants=()) -> None:
+        """W = [gate rows; up rows]: z[n, I] = act(x . gate^T) * (x . up^T), act = silu or the tanh form of gelu, or the clamped gate with
+        its constants (`ops.swiglu`).
         `scratch_fn()` gives a float32 [n, 2 I] buffer for the unfused path."""
         I = self.out_features // 2
         if self._tc(x) and z.dtype == torch.bfloat16:
-            ops.gemm_tc(x, self.weight, z, ops.SWIGLU + ops.GATE_ACTIVATIONS[activation], half_rows=I)
+            ops.gemm_tc(x, self.weight, z, ops.SWIGLU + ops.GATE_ACTIVATIONS[activation], half_rows=I, constants=constants or (0.0, 0.0))
         else:
             gate_up = scratch_fn()
             ops.gemm_f32(x, self.weight, gate_up, accumulate=False)
-            ops.swiglu(gate_up, z, activation)
+            ops.swiglu(gate_up, z, activation, constants or (0.0, 0.0))

@@ -140,13 +140,18 @@ class DecodeChain:
 class _StreamHolder:
     """The residual stream's buffer as the operations of a program see it."""
     _h, h_touched, _fresh, _stream = None, False, False, None
+    narrow = None                # the buffer that holds the residual stream once more as bfloat16, while it does
+
+    def note_narrow(self, buffer) -> None:
+        """`buffer` holds the stream's present rows as bfloat16. The note lapses as soon as an operation asks for the stream's buffer."""
+        self.narrow = buffer
 
     @property
     def h(self):
         """The buffer [max_rows, hidden] float32 that operations adding to the stream write into. A block that runs a sublayer on a branch
         puts the branch's buffer here meanwhile, and learns from `h_touched` whether any operation wrote into it (or only left partial
         sums pending). Asked for while the branch holds nothing yet (`set_fresh`), it is set to zero first."""
-        self.h_touched = True
+        self.h_touched, self.narrow = True, None
         if self._fresh:
             self._fresh = False
             self.add("branch", "sb_op_branch_clear", [self._h, self._h.shape[1]])

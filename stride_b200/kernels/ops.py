@@ -165,15 +165,16 @@ def rope_append(qkv: torch.Tensor, positions, slots, cos_sin, rotary_dim: int, q
                    cache_layer.stride(2), n, num_heads, num_kv_heads, head_dim, int(write_kv), int(values_from_keys), _stream()))
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}     # clamped: constants (limit, slope)
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out[n, I] = act(gate_up[:, :I]) * gate_up[:, I:], act = silu or the tanh form of gelu."""
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", constants=(0.0, 0.0)) -> None:
+    """out[n, I] = act(gate_up[:, :I]) * gate_up[:, I:], act = silu or the tanh form of gelu; or, "clamped" with constants (limit, slope),
+    g sigmoid(slope g) (u + 1) with g = min(gate, limit) and u = up within +-limit."""
     _cuda(gate_up, out)
-    lib, fn = _fn("elementwise", "sb_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    lib, fn = _fn("elementwise", "sb_swiglu_gated", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
     n, I = out.shape
-    _check(lib, fn(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), n, I, GATE_ACTIVATIONS[activation], _stream()))
+    _check(lib, fn(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), n, I, GATE_ACTIVATIONS[activation], *constants, _stream()))
 
 
 def cap_logits(logits: torch.Tensor, scale: float, cap: float) -> None:
@@ -243,7 +244,7 @@ def sample_temperature(logits, temperatures, seeds, lengths, tokens, values, sca
                    _ptr(scatter) if scatter_index is not None else 0, _stream()))
 
 
-STORE, ADD, SWIGLU, GEGLU_TANH = 0, 1, 2, 3     # GEGLU_TANH: SWIGLU with the tanh form of gelu on the gate
+STORE, ADD, SWIGLU, GEGLU_TANH, CLAMPED_GLU = 0, 1, 2, 3, 4     # SWIGLU with the tanh form of gelu on the gate; with the clamped gate
 
 
 def gemm_tc_splits(M: int, K: int) -> int:
@@ -262,7 +263,7 @@ def gemm_tc_partial_tokens() -> int:
 
 
 def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: int = STORE, splits: int = 1,
-            half_rows: int = 0) -> None:
+            half_rows: int = 0, constants=(0.0, 0.0)) -> None:
     """out = x . weight^T on the tcgen05 tensor cores; x [n, K] and weight [M, K] bfloat16.
 
     STORE: out float32 [n, M]. With splits > 1 (= gemm_tc_splits) and at most gemm_tc_partial_tokens() tokens, out is
@@ -270,15 +271,16 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: 
     ranges itself, in the same order, and out is [n, M].
     ADD: out float32 [n, M] += result (one range only).
     SWIGLU: weight is [2 I, K] (gate rows, then up rows) and out bfloat16 [n, I] = silu(x . gate^T) * (x . up^T).
+    GEGLU_TANH, CLAMPED_GLU: the same with another gate (`swiglu`; CLAMPED_GLU takes `constants`).
     """
     _cuda(x, weight, out)
     if x.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16:
         raise TypeError("gemm_tc takes bfloat16 operands")
-    want = torch.bfloat16 if epilogue in (SWIGLU, GEGLU_TANH) else torch.float32
+    want = torch.bfloat16 if epilogue in (SWIGLU, GEGLU_TANH, CLAMPED_GLU) else torch.float32
     if out.dtype != want:
         raise TypeError(f"gemm_tc epilogue {epilogue} writes {want}")
-    lib, fn = _fn("gemm_tc", "sb_gemm_tc", [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int,
-                                            c_int, c_int, c_int64, c_int, c_void_p])
+    lib, fn = _fn("gemm_tc", "sb_gemm_tc_gated", [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int,
+                                                  c_int, c_int, c_int64, c_int, c_float, c_float, c_void_p])
     n, K = x.shape
     M = weight.shape[0]
     if weight.shape[1] != K:
@@ -291,7 +293,7 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: 
         o2 = out[0] if out.dim() == 3 else out
         ldo, split_stride = o2.stride(0), 0
     _check(lib, fn(_ptr(x), x.stride(0), _ptr(weight), weight.stride(0), _ptr(out), ldo, n, M, K, epilogue, splits,
-                   split_stride, half_rows, _stream()))
+                   split_stride, half_rows, *constants, _stream()))
 
 
 def gemm_tc_status() -> int:

@@ -2,7 +2,7 @@ from .base import (Block, BranchScale, BuildEnv, CacheNeed, FeedForward, Mixer, 
                    register_part)
 from .context import ResidualStream, StepContext, Workspace
 from .spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry, TensorPlan
-from . import (attention, block, branch, ends, experts, gated_attention, gated_delta, hgrn2, lightning, masked_attention, mlp, norm,  # register the
+from . import (attention, block, branch, conv_attention, ends, experts, gated_attention, gated_delta, hgrn2, lightning, masked_attention, mlp, norm,  # register the
                parallel, reentry, retention, rglru, rope, sigmoid_attention, streams, token_side)                                            # built-in kinds
 from .model import DecoderModel
 

@@ -8,6 +8,9 @@ last projection adds into the branch or leaves its K ranges' partial sums pendin
 both into the stream in one pass (csrc/branch.cu) and leaves the branch zero again. A part that is several parts side by
 side may hand its members' branches over unfolded (`forward_sources` / `emit_sources`), so that one pass scales and adds them all.
 
+Blocks "postnorm" and "postnorm_mixer": no norm in front of a sublayer, it reads the residual itself (in the bfloat16 engine its rounding,
+which the fold in front stores beside the new rows), h += scale(mixer(h)), then (the first kind) h += scale(feed_forward(h)).
+
 "rmsnorm" (category "branch_scale" too): h += w * r / sqrt(mean(r^2) + eps), a norm on the sublayer's result, for designs that norm a
 sublayer on both sides; the same blocks, the same branches, one kernel that norms on the way."""
 from __future__ import annotations
@@ -15,6 +18,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
+from ..kernels.native import ImmediateProgram
 from .base import Block, BranchScale, register_part
 from .context import ResidualStream
 from .spec import TensorPlan
@@ -123,9 +127,10 @@ class BranchRMSNorm(BranchScale):
         (b, pb), cb = (sources[1][0].source(), sources[1][1]) if len(sources) > 1 else ((None, None), 1.0)
         ops.branch_norm_fold(stream.h, self.weight, self.eps, a=a, a_partials=pa, ca=ca, b=b, b_partials=pb, cb=cb)
 
-    def emit(self, program, sources):
+    def emit(self, program, sources, copy=None):
+        """`copy`: a bfloat16 buffer that the stream's new rows are stored in once more, for a sublayer that reads the stream itself."""
         program.need_folded("a norm behind a sublayer")
-        emit_fold(program, sources, self.weight, self.size, norm_eps=self.eps)
+        emit_fold(program, sources, self.weight, self.size, norm_eps=self.eps, copy=copy)
 
 
 ALWAYS = 1 << 30      # the limit of partial sums that are never added by the kernel that makes them, however many tokens a step has
@@ -136,9 +141,10 @@ def pending_limit(pending) -> int:
     return pending[3] if pending is not None and len(pending) > 3 else 0
 
 
-def emit_fold(program, sources, gain, width: int, norm_eps: float = None) -> None:
+def emit_fold(program, sources, gain, width: int, norm_eps: float = None, copy=None) -> None:
     """The operation that takes one or two branches (buffer or None, pending or None, constant) into the program's stream; with
-    `norm_eps` their sum is RMS-normed over its row before the gain."""
+    `norm_eps` their sum is RMS-normed over its row before the gain (and the new rows may go to a bfloat16 `copy` too). A branch's constant
+    may be a float32 tensor instead: a factor per row."""
     if not 1 <= len(sources) <= 2:
         raise ValueError("a fold takes one or two branches")
     (a, pa, ca), (b, pb, cb) = sources[0], sources[1] if len(sources) > 1 else (None, None, 1.0)
@@ -146,11 +152,12 @@ def emit_fold(program, sources, gain, width: int, norm_eps: float = None) -> Non
     if a is None and fa is None:
         raise ValueError("a branch that nothing wrote into")
     ints = [program.h, a, fa, Sa, program.few_tokens, b, fb, Sb, gain, gain.dtype if gain is not None else 0, width,
-            pending_limit(pa), pending_limit(pb)]
+            pending_limit(pa), pending_limit(pb), *(c if isinstance(c, torch.Tensor) else None for c in (ca, cb))]
+    ca, cb = (1.0 if isinstance(c, torch.Tensor) else c for c in (ca, cb))
     if norm_eps is None:
         program.add("branch", "sb_op_branch_fold", ints, [ca, cb])
     else:       # the branches' sum is RMS-normed over its row on the way
-        program.add("branch", "sb_op_branch_norm_fold", ints, [ca, cb, norm_eps])
+        program.add("branch", "sb_op_branch_norm_fold", [*ints, copy], [ca, cb, norm_eps])
 
 
 class _ScaledBlock(Block):
@@ -215,3 +222,62 @@ class PreNormScaledMixerBlock(_ScaledBlock):
 
     def emit(self, program, cache):
         self._emit_sublayer(program, self.mixer_norm, self.mixer, lambda f, x: f(program, x, cache), self.mixer_scale)
+
+
+class _PostNormBlock(Block):
+    graph_safe = True
+
+    def _input(self, program):
+        """The residual as a sublayer reads it: itself in the 32-bit engine, its bfloat16 rounding otherwise."""
+        if program.pending is not None:         # a block in front left partial sums
+            flat, S, _ = program.take_pending()
+            program.add("branch", "sb_op_stream_add", [program.h, flat, S, program.few_tokens, None, None, 0, program.h.shape[1]])
+        if self.env.act_dtype == torch.float32:
+            return program.h
+        if program.narrow is not None:
+            return program.narrow
+        h, ws = program.h, program.workspace
+        width = h.shape[1]
+        x = ws.get("block.x", ws.max_tokens, (width,), self.env.act_dtype)
+        program.add("elementwise", "sb_op_cast_columns", [h, width, 1, program.few_tokens, 0, width, x, x.dtype])
+        return x
+
+    def _emit_sublayer(self, program, part, run, scale):
+        ws = program.workspace
+        x = self._input(program)
+        if hasattr(part, "emit_sources"):
+            sources = run(part.emit_sources, x)
+        else:
+            branch = ws.get("postnorm.branch", ws.max_tokens, (program.h.shape[1],), torch.float32)
+            sources = [(*emit_on_branch(program, branch, lambda: run(part.emit, x), fresh=True), 1.0)]
+        copy = None
+        if self.env.act_dtype != torch.float32:
+            copy = ws.get("block.x", ws.max_tokens, (program.h.shape[1],), self.env.act_dtype)
+        scale.emit(program, sources, copy)
+        if copy is not None:
+            program.note_narrow(copy)
+
+    def kernel_libraries(self):
+        return super().kernel_libraries() | {"branch", "elementwise"}
+
+    def forward(self, ctx, stream, cache):
+        with ImmediateProgram(ctx, stream) as program:
+            self.emit(program, cache)
+
+
+@register_part("block", "postnorm")
+class PostNormBlock(_PostNormBlock):
+    ROLES = {"mixer": "mixer", "mixer_scale": "branch_scale", "feed_forward": "feed_forward", "feed_forward_scale": "branch_scale"}
+
+    def emit(self, program, cache):
+        self._emit_sublayer(program, self.mixer, lambda f, x: f(program, x, cache), self.mixer_scale)
+        self._emit_sublayer(program, self.feed_forward, lambda f, x: f(program, x), self.feed_forward_scale)
+
+
+@register_part("block", "postnorm_mixer")
+class PostNormMixerBlock(_PostNormBlock):
+    """The first half alone: a layer without a feed-forward."""
+    ROLES = {"mixer": "mixer", "mixer_scale": "branch_scale"}
+
+    def emit(self, program, cache):
+        self._emit_sublayer(program, self.mixer, lambda f, x: f(program, x, cache), self.mixer_scale)

@@ -16,7 +16,8 @@ Two parameters make other routed designs of it. `weights_from` "logits": the sto
 W_down (silu(W_gate x) * (W_up x)); its gate and up matrices lie one above the other in the side-by-side product.
 
 "table_experts": gated experts without a router, chosen by a stored table of token ids; the products run grouped, every expert on the rows
-that chose it (csrc/grouped_gemm.cu)."""
+that chose it (csrc/grouped_gemm.cu). "sigmoid_experts": the same grouped products behind a router, whose chosen scores are sigmoids taken as
+they are and multiply the experts' inputs."""
 from __future__ import annotations
 
 import torch
@@ -165,32 +166,29 @@ class RoutedFeedForward(FeedForward):
             self.down.emit_add(program, z, ws.raw("routed.down_partials", (self.down.partial_elems(T),), f32))
 
 
-@register_part("feed_forward", "table_experts")
-class TableExpertsFeedForward(FeedForward):
-    """Gated experts W_down (silu(W_gate x) * (W_up x)) chosen by the token alone: a stored table names `top` experts for every token id, each
-    with weight 1 / top; a shared expert of the same form may run for every token beside them. The step's (token, choice) pairs are sorted
-    by expert and every projection is one launch over the experts in use, each on its own rows (csrc/grouped_gemm.cu); the choices of a
-    token come back as `top` partial sums, which whoever takes the result in adds in their order, beside the shared expert's.
-    params: hidden_size, vocab_size, intermediate_size (of one expert), experts, top, shared (its intermediate size; 0: none).
-    tensors: table [vocab, top], gate, up, down (lists of names, one per expert), shared_gate, shared_up, shared_down."""
+class GroupedExpertsFeedForward(FeedForward):
+    """Gated experts W_down (silu(W_gate x) * (W_up x)) of which every token uses `top`, and perhaps a shared one of the same form: the
+    step's (token, choice) pairs are sorted by expert and every projection is one launch over the experts in use, each on its own rows
+    (csrc/grouped_gemm.cu); the choices of a token come back as `top` partial sums, which whoever takes the result in adds in their order.
+    Which experts a token uses is a subclass's business. params: hidden_size, intermediate_size (of one expert), experts, top, shared (the
+    shared expert's intermediate size; 0: none). tensors: gate, up, down (lists of names, one per expert), shared_gate, shared_up, shared_down."""
     graph_safe = True
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
         p = spec.params
-        self.hidden, self.vocab, self.intermediate = int(p["hidden_size"]), int(p["vocab_size"]), int(p["intermediate_size"])
+        self.hidden, self.intermediate = int(p["hidden_size"]), int(p["intermediate_size"])
         self.experts, self.top, self.shared_size = int(p["experts"]), int(p["top"]), int(p.get("shared", 0) or 0)
         if not 0 < self.top <= self.experts or self.experts > 1024:
-            raise ValueError(f"experts by table: {self.top} of {self.experts} experts (at most 1024)")
+            raise ValueError(f"grouped experts: {self.top} of {self.experts} experts (at most 1024)")
         t = spec.tensors
         self.shared = SwiGLU(PartSpec("gated", {"hidden_size": self.hidden, "intermediate_size": self.shared_size},
                                       {"gate": t["shared_gate"], "up": t["shared_up"], "down": t["shared_down"]}), env) if self.shared_size else None
-        self.table = self.gate_up = self.down = None
+        self.gate_up = self.down = None
         self.tensor_core = False
 
     def tensor_plan(self):
-        t = self.spec.tensors
-        plan = {t["table"]: TensorPlan((self.vocab, self.top), integer=True, below=self.experts)}
+        t, plan = self.spec.tensors, {}
         for name in (*t["gate"], *t["up"]):
             plan[name] = TensorPlan((self.intermediate, self.hidden))
         for name in t["down"]:
@@ -208,10 +206,6 @@ class TableExpertsFeedForward(FeedForward):
                 ws = [w.to(torch.float32) for w in ws]
             return torch.cat(ws, dim=0).contiguous()
 
-        self.table = tensors[t["table"]].contiguous()
-        low, high = int(self.table.min()), int(self.table.max())
-        if low < 0 or high >= self.experts:
-            raise ValueError(f"experts by table: '{t['table']}' names experts {low} .. {high} of {self.experts}")
         self.gate_up = one_below_the_other([name for pair in zip(t["gate"], t["up"]) for name in pair])      # [E (F gate rows, F up rows), hidden]
         self.down = one_below_the_other(t["down"])                                                          # [E hidden, F]
         self.tensor_core = (self.env.compute_dtype == torch.bfloat16 and self.gate_up.dtype == self.down.dtype == torch.bfloat16
@@ -232,17 +226,18 @@ class TableExpertsFeedForward(FeedForward):
             self.emit(program, x)
 
     def emit(self, program, x):
-        program.need_folded("experts by table")
+        program.need_folded("grouped experts")
         emit_fold(program, self.emit_sources(program, x), None, self.hidden)
 
-    def emit_sources(self, program, x):
-        """The result as branches with constants, left to the caller to add."""
+    def _emit_grouped(self, program, x, choice, vocab: int, pair_weight, scale: float) -> list:
+        """The chosen experts' and the shared expert's results as branches with constants. choice [vocab, top]: the experts of every token
+        id; with vocab 0, [tokens of the step, top]. pair_weight [top, tokens]: a factor on every pair's input, or None."""
         ws, E, top, F, W, tc = program.workspace, self.experts, self.top, self.intermediate, self.hidden, int(self.tensor_core)
         T, i32, act = ws.max_tokens, torch.int32, self.env.act_dtype
         order = ws.raw("experts.order", (T * top,), i32)
         tiles = ws.raw("experts.tiles", (3 * T * top + 1,), i32)
         lib = "grouped_gemm"
-        program.add(lib, "sb_op_expert_sort", [self.table, self.vocab, top, E, getattr(program, "sampled", None), order, tiles, tc])
+        program.add(lib, "sb_op_expert_sort", [choice, vocab, top, E, getattr(program, "sampled", None), order, tiles, tc])
         if tc:
             xs = ws.raw("experts.x", (T * top, W), act)
             program.add(lib, "sb_op_expert_gather", [x, x.stride(0), x.element_size(), order, top, xs, W])
@@ -250,11 +245,87 @@ class TableExpertsFeedForward(FeedForward):
             xs = x
         z = ws.raw("experts.z", (T * top, F), act)
         program.add(lib, "sb_op_expert_linear", [xs, xs.stride(0), xs.dtype, self.gate_up, self.gate_up.dtype, z, z.dtype, 2 * F, W, E, top, 1,
-                                                 order, tiles, tc])
+                                                 order, tiles, tc, pair_weight])
         out = ws.raw("experts.out", (T * top * W,), torch.float32)
         program.add(lib, "sb_op_expert_linear", [z, F, z.dtype, self.down, self.down.dtype, out, out.dtype, W, F, E, top, 0, order, tiles, tc])
-        sources = [(None, (out, top, W, ALWAYS), 1.0 / top)]
+        sources = [(None, (out, top, W, ALWAYS), scale)]
         if self.shared is not None:
             branch = ws.get("experts.shared", T, (W,), torch.float32)
             sources.append((*emit_on_branch(program, branch, lambda: self.shared.emit(program, x), fresh=True), 1.0))
         return sources
+
+
+@register_part("feed_forward", "sigmoid_experts")
+class SigmoidExpertsFeedForward(GroupedExpertsFeedForward):
+    """Grouped experts behind a router in 32-bit: z = W_r x, the `top` experts with the largest z are chosen, and the score of a chosen one,
+    s = sigmoid(z) as it is, multiplies the expert's input: sum of expert(s x). The shared expert's result may be multiplied by a gate per
+    token, sigmoid(W_sg x): one more row of the router's product.
+    params further: shared_gate (False by default). tensors further: router [experts, hidden], shared_sg [1, hidden]."""
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.shared_gate = bool(spec.params.get("shared_gate")) and self.shared_size > 0
+        self.router = None
+
+    def tensor_plan(self):
+        t, plan = self.spec.tensors, super().tensor_plan()
+        plan[t["router"]] = TensorPlan((self.experts, self.hidden))
+        if self.shared_gate:
+            plan[t["shared_sg"]] = TensorPlan((1, self.hidden))
+        return plan
+
+    def bind(self, tensors):
+        super().bind(tensors)
+        t = self.spec.tensors
+        rows = [tensors[t["router"]], *([tensors[t["shared_sg"]]] if self.shared_gate else [])]
+        if len({w.dtype for w in rows}) > 1:
+            rows = [w.to(torch.float32) for w in rows]
+        self.router = torch.cat(rows, dim=0).contiguous()
+
+    def weight_bytes(self):
+        return super().weight_bytes() + self.router.numel() * self.router.element_size()
+
+    def kernel_libraries(self):
+        return super().kernel_libraries() | {"gemm_f32"}
+
+    def emit_sources(self, program, x):
+        """The result as branches with constants, left to the caller to add."""
+        ws, E, top, f32 = program.workspace, self.experts, self.top, torch.float32
+        T, X = ws.max_tokens, self.router.shape[0]
+        logits = ws.get("experts.logits", T, (X,), f32)
+        program.add("gemm_f32", "sb_op_linear_f32", [x, x.dtype, x.stride(0), self.router, self.router.dtype, self.router.stride(0), logits, X, X,
+                                                     self.hidden, 0, 0])
+        choice = ws.raw("experts.choice", (T * top,), torch.int32)
+        weights = ws.raw("experts.weights", (T * top,), f32)
+        gate = ws.raw("experts.shared_gate", (T,), f32) if self.shared_gate else None
+        program.add("grouped_gemm", "sb_op_expert_choose", [logits, X, E, top, choice, weights, gate])
+        sources = self._emit_grouped(program, x, choice, 0, weights, 1.0)
+        if gate is not None:
+            sources[1] = (*sources[1][:2], gate)
+        return sources
+
+
+@register_part("feed_forward", "table_experts")
+class TableExpertsFeedForward(GroupedExpertsFeedForward):
+    """Grouped experts without a router, chosen by the token alone: a stored table names `top` experts for every token id, each with weight
+    1 / top. params further: vocab_size. tensors further: table [vocab, top]."""
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.vocab = int(spec.params["vocab_size"])
+        self.table = None
+
+    def tensor_plan(self):
+        return {self.spec.tensors["table"]: TensorPlan((self.vocab, self.top), integer=True, below=self.experts), **super().tensor_plan()}
+
+    def bind(self, tensors):
+        t = self.spec.tensors
+        self.table = tensors[t["table"]].contiguous()
+        low, high = int(self.table.min()), int(self.table.max())
+        if low < 0 or high >= self.experts:
+            raise ValueError(f"experts by table: '{t['table']}' names experts {low} .. {high} of {self.experts}")
+        super().bind(tensors)
+
+    def emit_sources(self, program, x):
+        """The result as branches with constants, left to the caller to add."""
+        return self._emit_grouped(program, x, self.table, self.vocab, None, 1.0 / self.top)

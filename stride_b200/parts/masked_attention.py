@@ -49,15 +49,15 @@ def _page_where(pages, table):
     return [table.shape[1], pages.shape[3], pages.stride(0), pages.stride(1) if pages.shape[1] > 1 else 0, pages.stride(2)]
 
 
-def _emit_attend(program, q, out, cache, slopes, sinks, H, G, D, Dv, window, keep_first, scale, tiles):
+def _emit_attend(program, q, out, cache, slopes, sinks, H, G, D, Dv, window, keep_first, scale, tiles, cap=0.0):
     pages, table = cache.pages, cache.block_table
     if tiles:
         program.add("masked_attention", "sb_op_masked_attention_tiles",
-                    [q, out, pages, table, *_page_where(pages, table), slopes, sinks, H, G, D, Dv, pages.shape[4], window, keep_first], [scale])
+                    [q, out, pages, table, *_page_where(pages, table), slopes, sinks, H, G, D, Dv, pages.shape[4], window, keep_first], [scale, cap])
     else:
         program.add("masked_attention", "sb_op_masked_attention",
                     [q, out, q.dtype, pages, table, *_page_where(pages, table), slopes, sinks, H, G, D, Dv, pages.shape[4], window, keep_first],
-                    [scale])
+                    [scale, cap])
 
 
 @register_part("mixer", "masked_attention")
