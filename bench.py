@@ -332,7 +332,7 @@ def _keralorn_config(width: int, ff: int, vocab: int, pairs: int, window: int) -
     """`pairs` times (windowed attention, lightning), each with a feed-forward, all inside one pass of the loop: the
     attention layer has the heads of the Llama 3.2 1B layer, the lightning layer 16 heads of 128 x 128."""
     att = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
-           "mixer": {"heads": width // 64, "kv_heads": width // 256, "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": window},
+           "mixer": {"heads": width // 64, "kv_heads": width // 256, "dim": 64, "vdim": 64, "scale": 0.125, **({"mask": {"size": window}} if window else {}),
                      "rot": {"dims": 32, "base": 500000.0, "scaling": {"factor": 32.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
     heads = width // 128
     lig = {"type": "lightning", "mlp": {"kind": "dense", "ff": ff},
@@ -399,6 +399,19 @@ def _viperax_config(width: int, ff: int, vocab: int, pairs: int, window: int) ->
             "logit_scale": 0.5, "logit_softcap": 15.0, "layers": layers}
 
 
+def _mezadra_config(width: int, ff: int, vocab: int, pairs: int, dense: bool = False) -> dict:
+    """`pairs` times (attention behind a short convolution, lightning), heads as in the Keralorn configuration; the attention layers have a
+    clamped dense feed-forward, the lightning layers eight experts of ff / 4, one per token, and a gated shared one (`dense`: all are dense)."""
+    att = {"type": "attention", "mlp": {"kind": "dense", "ff": ff, "limit": 7.0},
+           "mixer": {"heads": width // 64, "kv_heads": width // 256, "dim": 64, "vdim": 64, "scale": 0.125, "conv": 4, "softcap": 30.0, "v_mix": True,
+                     "rot": {"dims": 32, "base": 500000.0}}}
+    heads = width // 128
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 8, "top": 1}, "shared": {"ff": ff // 4}}
+    lig = {"type": "lightning", "mlp": att["mlp"] if dense else moe,
+           "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-3 - 5.0 * h / max(heads - 1, 1)) for h in range(heads)]}}
+    return {"architecture": "Mezadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "layers": [att, lig] * pairs}
+
+
 def design_compare(a) -> int:
     """Keralorn at layer sizes of a real model beside LlamaForCausalLM with as many layers of the same width, heads and
     feed-forward (random weights, bfloat16 engine): a prompt of 2,048 tokens in one step, decode steps at batch 8 and 64
@@ -423,9 +436,15 @@ def design_compare(a) -> int:
         configs = {"viperax": _viperax_config(width, ff, vocab, pairs, 1024), "pusisun": _pusisun_config(width, ff, vocab, pairs, 1024),
                    "viperax_width_4096": _viperax_config(4096, 14336, vocab, pairs, 1024),
                    "pusisun_width_4096": _pusisun_config(4096, 14336, vocab, pairs, 1024)}
+    if a.design == "mezadra":      # beside the closest design (softmax attention alternating with the same linear attention), at two widths; with experts too
+        configs = {}
+        for w, f in ((2048, 8192), (4096, 14336)):
+            tail = "" if w == width else f"_width_{w}"
+            configs.update({"mezadra_dense" + tail: _mezadra_config(w, f, vocab, pairs, dense=True), "keralorn" + tail: _keralorn_config(w, f, vocab, pairs, 0),
+                            "mezadra_experts" + tail: _mezadra_config(w, f, vocab, pairs)})
     gen = torch.Generator().manual_seed(3)
     out = {"design": a.design, "beside": {"keralorn": "LlamaForCausalLM", "ganupel": "Keralorn, LlamaForCausalLM", "pusisun": "Ganupel, LlamaForCausalLM",
-                                          "sitivik": "Ganupel, LlamaForCausalLM", "viperax": "Pusisun"}[a.design], "width": width, "ff": ff, "layers": layers, "vocab": vocab,
+                                          "sitivik": "Ganupel, LlamaForCausalLM", "viperax": "Pusisun", "mezadra": "Keralorn"}[a.design], "width": width, "ff": ff, "layers": layers, "vocab": vocab,
            "dtype": "bf16", "data": "synthetic (random weights and tokens)", "peaks": pk,
            "l2": "weights and caches of a step exceed the 126 MB L2; the kernel timings flush L2 between launches"}
     flush = torch.empty(160 << 20, dtype=torch.uint8, device="cuda")
@@ -503,9 +522,9 @@ def design_compare(a) -> int:
         del eng
         torch.cuda.empty_cache()
 
-    if a.design in ("ganupel", "pusisun", "sitivik", "viperax"):
+    if a.design in ("ganupel", "pusisun", "sitivik", "viperax", "mezadra"):
         out["kernels"] = {"ganupel": _ganupel_kernels, "pusisun": _pusisun_kernels, "sitivik": _sitivik_kernels,
-                          "viperax": _viperax_kernels}[a.design](timed, pk, width, ff)
+                          "viperax": _viperax_kernels, "mezadra": _mezadra_kernels}[a.design](timed, pk, width, ff)
         out["clocks"] = clocks.stop()
         print(json.dumps(out))
         return 0
@@ -1038,6 +1057,106 @@ def _viperax_kernels(timed, pk: dict, width: int, ff: int) -> dict:
     return kern
 
 
+def _mezadra_kernels(timed, pk: dict, width: int, ff: int) -> dict:
+    """Mezadra's own kernels alone (L2 flushed between launches), each beside the like kernel of Keralorn (experts: of Viperax)."""
+    import torch
+    from stride_b200.kernels import ops
+    from stride_b200.kernels.native import ImmediateProgram
+    from stride_b200.parts import Workspace
+    from stride_b200.parts.context import step_context
+    dev, kern, f32, bf, i32 = "cuda", {}, torch.float32, torch.bfloat16, torch.int32
+    hbm = pk["hbm_gbs"] * 1e9
+
+    def record(label, ms, moved=None, flops=None, **more):
+        r = {"ms": round(ms, 4)}
+        if moved is not None:
+            r.update(gb_s=round(moved / ms / 1e6, 1), hbm_fraction_of_measured=round(moved / (ms * 1e-3) / hbm, 3))
+        if flops is not None:
+            r.update(tflops=round(flops / ms / 1e9, 2), fraction_of_measured_bf16=round(flops / ms / 1e9 / pk["bf16_tflops"], 4))
+        r.update(more)
+        kern[label] = r
+
+    ws = Workspace(dev, 2048)
+    H, G, D, taps, rot, page = width // 64, width // 256, 64, 4, 32, 64
+    C = (H + 2 * G) * D
+    E, F = 8, ff // 4
+    rand = lambda *shape: torch.randn(*shape, device=dev)
+    gain = torch.ones(width, device=dev)
+    w_up, w_down = (rand(E * 2 * F, width) * 0.02).to(bf), (rand(E * width, F) * 0.02).to(bf)
+    router = (rand(E + 1, width) * 0.02).to(bf)
+    dense = (rand(2 * ff, width) * 0.02).to(bf)
+    cs, conv = torch.rand(4096, rot // 2, 2, device=dev), rand(taps, C)
+    sinks = torch.zeros(H, device=dev)
+    for label, entries, length, past in (("prefill_2048", 1, 2048, 0), ("decode_b64", 64, 1, 1500), ("decode_b8", 8, 1, 1500)):
+        n, per = entries * length, (past + length + page - 1) // page
+        ctx = step_context([(e, length, past) for e in range(entries)], ws, bf, rows=2048)
+        program = ImmediateProgram(ctx, None)
+        op = lambda library, function, ints, floats=(): program.prepared(library, function, ints, floats)
+        block = torch.arange(entries * per, dtype=i32, device=dev).view(entries, per)
+        pages = rand(entries * per + 1, 2, G, page, D).to(bf)
+        where = [pages, block, per, page, pages.stride(0), pages.stride(1), pages.stride(2)]
+        P = 1 if n > 512 else ops.gemm_tc_splits(C, width)          # K ranges of the projection in front, as buffers in steps of few tokens
+        proj, q, kept = rand(P * n * C), torch.empty(n, H * D, dtype=bf, device=dev), rand(n, G * D)
+        state = torch.zeros(entries, (taps - 1) * C, device=dev)
+        ms = timed(op("short_conv", "sb_op_conv_qkv", [proj, C, P, 512, conv, taps, state, (taps - 1) * C, cs, rot, 1, kept, 2, q, bf, *where, H, G, D, D, D], [1e-5, 0.5]),
+                   5, clear=True)
+        record("conv_qkv_" + label, ms, n * C * (4.0 * P + 2.0) + n * G * D * 4.0 + entries * (taps - 1) * C * 8.0)
+        qkv = proj.view(P, n, C)
+        ms = timed(lambda: ops.rope_append(qkv, ctx.positions, ctx.slots, cs, rot, q, pages, block, H, G, D), 5, clear=True)
+        record("keralorn_rope_append_" + label, ms, n * C * (4.0 * P + 2.0))
+        out = torch.empty(n, H * D, dtype=bf, device=dev)
+        plan = program.plan(H // G, 128, 1, -1)
+        keys = sum(past + t + 1 for t in range(length)) * entries
+        for name, floats, extra in (("attention_capped_with_sinks_", [0.125, 30.0], sinks), ("keralorn_attention_", [0.125, 0.0], None)):
+            if length > 1:
+                ms = timed(op("attention_tc5", "sb_op_attention_tc5", [q, out, pages, pages.shape[0], *where[1:], H, G, D, 0, plan, extra], floats), 5, clear=True)
+                record(name + label, ms, None, 4.0 * keys * H * D)
+            else:
+                need = ops.attention_tc_scratch
+                scratch = program.growing_buffer("attn.scratch", f32, 0, lambda step: need(step.plan[plan].items, G, step.plan[plan].chunks, D))
+                counters = torch.zeros(2048 * G, dtype=i32, device=dev)
+                ms = timed(op("attention_tc", "sb_op_attention_tc", [q, out, *where, scratch, 0, counters, H, G, D, 0, plan, 1, None, 0, 1, 0, None, extra], floats), 5,
+                           clear=True)
+                record(name + label, ms, entries * (past + 1) * G * D * 4.0 + n * H * D * 4.0)
+        # between two sublayers: the norm on a result with the second output; Keralorn's layer norm in front of one
+        P = 1 if n > 512 else 8
+        h, parts, two, x = rand(n, width), rand(P, n, width), rand(n, width), torch.empty(n, width, dtype=bf, device=dev)
+        fold = lambda b, factor: op("branch", "sb_op_branch_norm_fold", [h, None, parts, P, 512, b, None, 1, gain, f32, width, 0, 0, None, factor, x], [1.0, 1.0, 1e-5])
+        ms = timed(fold(None, None), 5, clear=True)
+        record("norm_fold_" + label, ms, n * width * (10.0 + 4.0 * P))
+        factor = rand(n)
+        ms = timed(fold(two, factor), 5, clear=True)
+        record("norm_fold_two_sources_" + label, ms, n * width * (18.0 + 4.0 * P))
+        bias = torch.zeros(width, device=dev)
+        ms = timed(lambda: ops.layernorm(h, gain, bias, 1e-5, x, partials=parts), 5, clear=True)
+        record("keralorn_layernorm_" + label, ms, n * width * (10.0 + 4.0 * P))
+        # the dense feed-forward's first product with the clamped gate; Keralorn's with the tanh form of gelu
+        xe = rand(n, width).to(bf)
+        zd = torch.empty(n, ff, dtype=bf, device=dev)
+        for name, mode in (("clamped_gate_up_", 5), ("keralorn_gelu_gate_up_", 4)):
+            ms = timed(op("gemm_tc", "sb_op_linear_tc", [xe, width, dense, width, zd, 2 * ff, width, mode, 1, 0], [7.0, 1.702]), 5, clear=True)
+            record(name + label, ms, dense.numel() * 2.0 + n * (width + ff) * 2.0, 4.0 * n * ff * width)
+        # experts: the router's product and choice, then the grouped products with and without weights on their inputs
+        logits, choice, weights, gate = torch.empty(n, E + 1, device=dev), torch.empty(n, dtype=i32, device=dev), torch.empty(n, device=dev), torch.empty(n, device=dev)
+        ms = timed(op("gemm_f32", "sb_op_linear_f32", [xe, bf, width, router, bf, width, logits, E + 1, E + 1, width, 0, 0]), 5, clear=True)
+        record("router_product_" + label, ms, n * width * 2.0)
+        ms = timed(op("grouped_gemm", "sb_op_expert_choose", [logits, E + 1, E, 1, choice, weights, gate]), 5, clear=True)
+        record("expert_choose_" + label, ms, n * (E + 1) * 4.0 + n * 12.0)
+        order, tiles = torch.empty(n, dtype=i32, device=dev), torch.empty(3 * n + 1, dtype=i32, device=dev)
+        xs, z, y = (torch.empty(n, k, dtype=t, device=dev) for k, t in ((width, bf), (F, bf), (width, f32)))
+        used = len(set(choice.tolist()))
+        ms = timed(op("grouped_gemm", "sb_op_expert_sort", [choice, 0, 1, E, None, order, tiles, 1]), 5, clear=True)
+        record("expert_sort_" + label, ms, n * 8.0)
+        ms = timed(op("grouped_gemm", "sb_op_expert_gather", [xe, width, 2, order, 1, xs, width]), 5, clear=True)
+        record("expert_gather_" + label, ms, n * width * 4.0)
+        for name, w in (("expert_gate_up_weighted_", weights), ("viperax_expert_gate_up_", None)):
+            ms = timed(op("grouped_gemm", "sb_op_expert_linear", [xs, width, bf, w_up, bf, z, bf, 2 * F, width, E, 1, 1, order, tiles, 1, w]), 5, clear=True)
+            record(name + label, ms, used * 2 * F * width * 2.0 + n * (width + F) * 2.0, 4.0 * n * F * width, experts_in_use=used)
+        ms = timed(op("grouped_gemm", "sb_op_expert_linear", [z, F, bf, w_down, bf, y, f32, width, F, E, 1, 0, order, tiles, 1, None]), 5, clear=True)
+        record("expert_down_" + label, ms, used * F * width * 2.0 + n * (F * 2.0 + width * 4.0), 2.0 * n * F * width, experts_in_use=used)
+    return kern
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1048,10 +1167,10 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--shape", default="1b", choices=sorted(SHAPES), help="1b: the decode step (default); 3b, 8b: serving runs")
     ap.add_argument("--skip-points", action="store_true", help="skip the batch 1 / 64, float32 and prefill measurements")
-    ap.add_argument("--design", default="", choices=["", "keralorn", "ganupel", "pusisun", "sitivik", "viperax"],
+    ap.add_argument("--design", default="", choices=["", "keralorn", "ganupel", "pusisun", "sitivik", "viperax", "mezadra"],
                     help="keralorn: prefill and decode of that design beside a Llama of equal layer sizes, and its own kernels alone; "
                          "ganupel: the same beside Keralorn and Llama; pusisun: the same beside Ganupel and Llama; "
-                         "viperax: the same beside Pusisun, at two widths")
+                         "viperax: the same beside Pusisun, at two widths; mezadra: the same beside Keralorn, at two widths")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)

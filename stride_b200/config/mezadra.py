@@ -88,7 +88,7 @@ class MezadraConfig:
                         raise ConfigError(f"config.json: '{mw}rot.dims' {dims} must be even and at most dim {dim}")
                     fields.update(rot_dims=dims, rot_base=_get(m["rot"], "base", mw + "rot.", float, True))
                 first = next((k for k in layers if k.v_mix), None)
-                if fields["v_mix"] and first is not None and (first.kv_heads, first.vdim) != (kv, vdim):
+                if fields["v_mix"] and first is not None and first.kv_heads * first.vdim != kv * vdim:
                     raise ConfigError(f"config.json: '{mw}v_mix': values of {kv} x {vdim} cannot be mixed with the first such layer's "
                                       f"{first.kv_heads} x {first.vdim}")
             elif kind == "lightning":

@@ -12,6 +12,9 @@
 //   fold   (m, l, o) <- (m_t, l_t, o_t): m' = max(m, m_t), a = ex2(m - m'), b = ex2(m_t - m'),
 //          l = fma(l, a, l_t * b), o = fma(o, a, o_t * b). The empty state is (-inf, 0, 0).
 //
+// Designs that cap their scores softly, C tanh(scale s / C): every raw score becomes t = tanh(scale s / C) first, and c is C * log2(e).
+// A sink (a term exp(sink) in the denominator, without key and value) joins the finished row: l + ex2(sink log2(e) - m) in place of l.
+//
 // tcgen05.mma (kind::f16) and mma.sync m16n8k16 give the same bits for the same products in the same order of
 // K steps on this hardware (checked by the tests), which is what lets kernels built on either share this.
 #pragma once
@@ -66,6 +69,14 @@ __device__ __forceinline__ FoldFactors fold_factors(float m, float m_t) {
 __device__ __forceinline__ float fold_value(float v, float v_t, const FoldFactors& f) {
   return __fmaf_rn(v, f.a, __fmul_rn(v_t, f.b));
 }
+// tanh(scale s / C) with k = 2 log2(e) scale / C: 1 - 2 / (1 + 2^(k s)), by the hardware's approximations of 2^x and of the reciprocal (an
+// infinite power gives 1, a vanishing one -1).
+__device__ __forceinline__ float capped_score(float s, float k) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(__fadd_rn(1.0f, ex2(__fmul_rn(s, k)))));
+  return __fmaf_rn(-2.0f, r, 1.0f);
+}
+__device__ __forceinline__ float with_sink(float l, float m, float sink) { return __fadd_rn(l, ex2(__fmaf_rn(sink, kLog2e, -m))); }
 __device__ __forceinline__ float finish(float o, float l) { return __fmul_rn(o, __frcp_rn(l)); }
 
 }  // namespace attn

@@ -44,7 +44,8 @@ constexpr int kDecodeCtas64 = SB_DECODE_CTAS64;   // CTAs of the decode kernel p
 
 
 // ------------------------------------------------------------------ prompt portions
-template <int D>
+// EXTRA (here and below): scores may be capped and rows may have sinks.
+template <int D, bool EXTRA>
 __global__ void __launch_bounds__(128) attn_chunk_kernel(const AttnTcParams p) {
   constexpr int LD = D + 8, CH = D / 8;
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -122,7 +123,7 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(const AttnTcParams p) {
       // every row of this warp that is in use sees every key of the tile: nothing to mask
       const bool full = warp_pos_lo >= 0 && kt * kKeys + kKeys - 1 <= warp_pos_lo &&
                         kt * kKeys >= (p.window > 0 ? warp_pos_hi - p.window + 1 : 0);
-      tile_partial<D>(s, o_t, m_t, l_t, kt * kKeys, row_pos, row_lo, p.scale_log2, sV + buf * 64 * LD, lane, full);
+      tile_partial<D>(s, o_t, m_t, l_t, kt * kKeys, row_pos, row_lo, p.scale_log2, sV + buf * 64 * LD, lane, full, EXTRA ? p.cap_k : 0.0f);
       fold_rows<D>(m_c, l_c, o_c, m_t, l_t, o_t);
     }
     if ((kt + 1) % (kChunk / kKeys) == 0 || kt == kt1) {
@@ -152,6 +153,7 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(const AttnTcParams p) {
     const int r = warp * 16 + gid + 8 * h;
     const int pi = div_g(p, r), hh = r - pi * G;
     if (pi < npos) {
+      if (EXTRA && p.sinks != nullptr) l_r[h] = with_sink(l_r[h], m_r[h], p.sinks[g * G + hh]);
       const float* row = sT + r * D + tq * 2;
       bf16* dst = p.out + (static_cast<int64_t>(row0 + pi) * p.Hq + g * G + hh) * D;
 #pragma unroll
@@ -170,7 +172,7 @@ struct BlockEnv {
   __device__ __forceinline__ void sync() { __syncthreads(); }
   __device__ __forceinline__ void wait_inputs() { sb::grid_dependency_wait(); }
 };
-template <int D, bool FUSED, bool CLUSTER>
+template <int D, bool FUSED, bool CLUSTER, bool EXTRA>
 __global__ void __launch_bounds__(128, FUSED ? 3 : (D == 64 ? kDecodeCtas64 : 3)) attn_decode_kernel(const AttnTcParams p) {
   extern __shared__ __align__(128) uint8_t smem_tiles[];
   __shared__ int is_last_s;
@@ -180,7 +182,7 @@ __global__ void __launch_bounds__(128, FUSED ? 3 : (D == 64 ? kDecodeCtas64 : 3)
   // cluster is the grid's z extent, so the rank is the chunk)
   static_assert((4 * 16 * (D + 2) + decode_record_floats<D>()) * sizeof(float) <= 4 * 64 * D * sizeof(bf16), "the record must fit over the tiles");
   float* record = CLUSTER ? reinterpret_cast<float*>(smem_tiles) + 4 * 16 * (D + 2) : nullptr;
-  decode_unit<D, FUSED, CLUSTER>(p, blockIdx.x, blockIdx.y, blockIdx.z, smem_tiles, &is_last_s, threadIdx.x, env, record);
+  decode_unit<D, FUSED, CLUSTER, EXTRA>(p, blockIdx.x, blockIdx.y, blockIdx.z, smem_tiles, &is_last_s, threadIdx.x, env, record);
 }
 
 template <int D>
@@ -197,7 +199,7 @@ __global__ void __launch_bounds__(D) attn_combine_kernel(const AttnTcParams p) {
   const int64_t rec0 = (static_cast<int64_t>(item) * p.Hkv + g) * p.chunks;
   for (int r = 0; r < L * G; ++r)
     p.out[(static_cast<int64_t>(first_row + r / G) * p.Hq + g * G + r % G) * D + d] =
-        __float2bfloat16_rn(fold_chunks<D>(p.part_o, p.part_ml, rec0, c0, c1, r, d));
+        __float2bfloat16_rn(fold_chunks<D>(p.part_o, p.part_ml, rec0, c0, c1, r, d, p.sinks != nullptr ? p.sinks + g * G + r % G : nullptr));
 }
 
 // The same fold for long contexts (tens to hundreds of chunks an entry), where the requests for the records and the
@@ -217,7 +219,7 @@ __global__ void __launch_bounds__(kStreamThreads) attn_combine_stream_kernel(con
   extern __shared__ __align__(16) float stages[];   // [2][stage_floats]
   __shared__ float before[kStreamChunks][16];        // [chunk of the stage][row]: the row's maximum before the chunk
   __shared__ float factor_a[kStreamChunks][16];      // a of (chunk, row); 1 where the row sees no key of the chunk
-  __shared__ float l_rows[16];
+  __shared__ float l_rows[16], m_rows[16];
   sb::grid_launch_dependents();
   const int item = blockIdx.x, g = blockIdx.y, d0 = blockIdx.z * kStreamSlice;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -331,7 +333,13 @@ __global__ void __launch_bounds__(kStreamThreads) attn_combine_stream_kernel(con
     }
     __syncthreads();   // this stage is requested again in the next round; `before` and `factor_a` are rewritten
   }
-  if (r_c < rows && j_c == kStreamSlice / 2) l_rows[r_c] = o0;
+  if (p.sinks != nullptr) {
+    const int r = warp + lane * (kStreamThreads / 32);
+    if (r < rows) m_rows[r] = m_row;
+    __syncthreads();
+  }
+  if (r_c < rows && j_c == kStreamSlice / 2)
+    l_rows[r_c] = p.sinks != nullptr ? with_sink(o0, m_rows[r_c], p.sinks[g * G + r_c - div_g(p, r_c) * G]) : o0;
   __syncthreads();
   if (r_c < rows && j_c < kStreamSlice / 2) {
     const int pi = div_g(p, r_c);
@@ -346,18 +354,18 @@ __global__ void __launch_bounds__(kStreamThreads) attn_combine_stream_kernel(con
 constexpr int kStreamFoldChunks = 32;
 constexpr size_t kStreamStageBytes = 40 * 1024;
 
-template <int D>
+template <int D, bool EXTRA>
 int launch(const AttnTcParams& p, int n_tiles, int n_items, cudaStream_t stream) {
   constexpr int LD = D + 8;
   if (n_tiles > 0) {
     const size_t smem = static_cast<size_t>(5) * 64 * LD * sizeof(bf16) + static_cast<size_t>(64) * D * sizeof(float);
     static sb::DeviceOnce once;
     if (once.needed()) {
-      if (cudaFuncSetAttribute(attn_chunk_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      if (cudaFuncSetAttribute(attn_chunk_kernel<D, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return sb::fail("sb_attention_tc: cannot raise the shared memory limit");
       once.done();
     }
-    sb::launch_pdl(attn_chunk_kernel<D>, dim3(n_tiles, p.Hkv), dim3(128), smem, stream, p);
+    sb::launch_pdl(attn_chunk_kernel<D, EXTRA>, dim3(n_tiles, p.Hkv), dim3(128), smem, stream, p);
   }
   if (n_items > 0) {
     // queries and the warps' tiles (keys and values, or one for both in turn); the results (4 x 16 x (D + 2) floats) reuse the tiles
@@ -366,11 +374,12 @@ int launch(const AttnTcParams& p, int n_tiles, int n_items, cudaStream_t stream)
     static_assert(4 * 64 * D * sizeof(bf16) >= 4 * 16 * (D + 2) * sizeof(float), "the results must fit over the tiles");
     static sb::DeviceOnce once;
     if (once.needed()) {
-      if (cudaFuncSetAttribute(attn_decode_kernel<D, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
-          cudaFuncSetAttribute(attn_decode_kernel<D, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_fused) != cudaSuccess ||
-          cudaFuncSetAttribute(attn_decode_kernel<D, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
-          cudaFuncSetAttribute(attn_decode_kernel<D, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_fused) != cudaSuccess)
-        return sb::fail("sb_attention_tc: cannot raise the shared memory limit");
+      bool ok = cudaFuncSetAttribute(attn_decode_kernel<D, false, false, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess &&
+                cudaFuncSetAttribute(attn_decode_kernel<D, false, true, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
+      if constexpr (!EXTRA)
+        ok = ok && cudaFuncSetAttribute(attn_decode_kernel<D, true, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_fused) == cudaSuccess &&
+             cudaFuncSetAttribute(attn_decode_kernel<D, true, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_fused) == cudaSuccess;
+      if (!ok) return sb::fail("sb_attention_tc: cannot raise the shared memory limit");
       once.done();
     }
     AttnTcParams pd = p;
@@ -384,14 +393,15 @@ int launch(const AttnTcParams& p, int n_tiles, int n_items, cudaStream_t stream)
     // launch run at once: 128 entries x 8 heads x 3 chunks 83 us with records in global memory, 91 us in clusters)
     const bool cluster = pd.counters != nullptr && p.chunks >= 2 && p.chunks <= 8 &&
                          (p.chunks == 2 || static_cast<long long>(n_items) * p.Hkv * p.chunks <= 2ll * sb::sm_count());
-    if (cluster) {
-      const dim3 shape(1, 1, p.chunks);
-      if (p.qkv != nullptr) sb::launch_pdl_cluster(attn_decode_kernel<D, true, true>, grid, dim3(128), smem_fused, stream, shape, pd);
-      else sb::launch_pdl_cluster(attn_decode_kernel<D, false, true>, grid, dim3(128), smem, stream, shape, pd);
-    } else if (p.qkv != nullptr) {
-      sb::launch_pdl(attn_decode_kernel<D, true, false>, grid, dim3(128), smem_fused, stream, pd);
+    const dim3 shape(1, 1, p.chunks);
+    if (p.qkv != nullptr) {
+      if constexpr (EXTRA) return sb::fail("sb_attention_tc: capped scores and sinks go with queries that are ready");
+      else if (cluster) sb::launch_pdl_cluster(attn_decode_kernel<D, true, true, false>, grid, dim3(128), smem_fused, stream, shape, pd);
+      else sb::launch_pdl(attn_decode_kernel<D, true, false, false>, grid, dim3(128), smem_fused, stream, pd);
+    } else if (cluster) {
+      sb::launch_pdl_cluster(attn_decode_kernel<D, false, true, EXTRA>, grid, dim3(128), smem, stream, shape, pd);
     } else {
-      sb::launch_pdl(attn_decode_kernel<D, false, false>, grid, dim3(128), smem, stream, pd);
+      sb::launch_pdl(attn_decode_kernel<D, false, false, EXTRA>, grid, dim3(128), smem, stream, pd);
     }
     if (stream_fold) {
       // two stages, each with room for all chunks (of 16 rows, in whole groups of eight) if that fits
@@ -432,7 +442,8 @@ int attention_tc_impl(const void* q, void* out, const void* k_base, const int32_
                       int page_size, int64_t page_stride, int64_t v_offset, int64_t head_stride,
                       const int32_t* meta, int meta_stride, const int32_t* work, int n_tiles, int n_items,
                       int chunks, float* scratch, int* counters, int Hq, int Hkv, int D, int window, float scale,
-                      const float* qkv, int n_partials, int64_t partial_stride, const float* cos_sin, cudaStream_t stream) {
+                      const float* qkv, int n_partials, int64_t partial_stride, const float* cos_sin, float cap, const float* sinks,
+                      cudaStream_t stream) {
   if (n_tiles <= 0 && n_items <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16)
     return sb::fail("sb_attention_tc: group ratio %d/%d is not supported (1..16)", Hq, Hkv);
@@ -461,7 +472,9 @@ int attention_tc_impl(const void* q, void* out, const void* k_base, const int32_
   for (int r = 0; r < 64; ++r)
     if (((r * p.g_mul) >> 16) != r / (Hq / Hkv)) return sb::fail("sb_attention_tc: the row arithmetic does not hold for %d/%d heads", Hq, Hkv);
   p.window = window;
-  p.scale_log2 = scale * kLog2e;
+  p.scale_log2 = (cap > 0.0f ? cap : scale) * kLog2e;
+  p.cap_k = cap > 0.0f ? 2.0f * kLog2e * scale / cap : 0.0f;
+  p.sinks = sinks;
   p.chunks = chunks;
   p.part_o = scratch;
   p.part_ml = scratch + static_cast<int64_t>(n_items) * Hkv * chunks * 16 * D;
@@ -470,8 +483,9 @@ int attention_tc_impl(const void* q, void* out, const void* k_base, const int32_
   p.n_partials = n_partials;
   p.partial_stride = partial_stride;
   p.cos_sin = cos_sin;
-  if (D == 64) return launch<64>(p, n_tiles, n_items, stream);
-  if (D == 128) return launch<128>(p, n_tiles, n_items, stream);
+  const bool extra = cap > 0.0f || sinks != nullptr;
+  if (D == 64) return extra ? launch<64, true>(p, n_tiles, n_items, stream) : launch<64, false>(p, n_tiles, n_items, stream);
+  if (D == 128) return extra ? launch<128, true>(p, n_tiles, n_items, stream) : launch<128, false>(p, n_tiles, n_items, stream);
   return sb::fail("sb_attention_tc: head_dim %d has no tensor-core kernel (64 or 128)", D);
 }
 }  // namespace
@@ -482,7 +496,16 @@ SB_EXPORT int sb_attention_tc(const void* q, void* out, const void* k_base, cons
                               int chunks, float* scratch, int* counters, int Hq, int Hkv, int D, int window, float scale,
                               cudaStream_t stream) {
   return attention_tc_impl(q, out, k_base, block_table, max_pages, page_size, page_stride, v_offset, head_stride, meta, meta_stride,
-                           work, n_tiles, n_items, chunks, scratch, counters, Hq, Hkv, D, window, scale, nullptr, 0, 0, nullptr, stream);
+                           work, n_tiles, n_items, chunks, scratch, counters, Hq, Hkv, D, window, scale, nullptr, 0, 0, nullptr, 0.0f, nullptr, stream);
+}
+
+// The same with scores capped softly at `cap` (0: not capped) and a sink per query head (float32 [Hq], or null).
+SB_EXPORT int sb_attention_tc_extra(const void* q, void* out, const void* k_base, const int32_t* block_table, int max_pages, int page_size,
+                                    int64_t page_stride, int64_t v_offset, int64_t head_stride, const int32_t* meta, int meta_stride,
+                                    const int32_t* work, int n_tiles, int n_items, int chunks, float* scratch, int* counters, int Hq, int Hkv,
+                                    int D, int window, float scale, float cap, const float* sinks, cudaStream_t stream) {
+  return attention_tc_impl(q, out, k_base, block_table, max_pages, page_size, page_stride, v_offset, head_stride, meta, meta_stride,
+                           work, n_tiles, n_items, chunks, scratch, counters, Hq, Hkv, D, window, scale, nullptr, 0, 0, nullptr, cap, sinks, stream);
 }
 
 // The decode kernel with the rotation and the append fused in, for a step whose entries all fit it (length * (Hq / Hkv)
@@ -500,7 +523,7 @@ SB_EXPORT int sb_attention_decode_rope(const float* qkv, int n_partials, int64_t
   if ((reinterpret_cast<uintptr_t>(cos_sin) & 7) != 0) return sb::fail("sb_attention_decode_rope: cos_sin must be 8-byte aligned");
   return attention_tc_impl(out, out, k_base, block_table, max_pages, page_size, page_stride, v_offset, head_stride, meta, meta_stride,
                            items, 0, n_items, chunks, scratch, counters, Hq, Hkv, D, window, scale, qkv, n_partials, partial_stride,
-                           cos_sin, stream);
+                           cos_sin, 0.0f, nullptr, stream);
 }
 
 
@@ -559,7 +582,7 @@ SB_EXPORT int sb_attention_decode_noalloc(const void* q, void* out, const void* 
 //    9 where the scratch buffer is noted (two int64 on the host: its device address and its size in floats; the engine
 //    enlarges the buffer before a step that needs more), 10 unused, 11 counters, 12 Hq, 13 Hkv, 14 D, 15 window, 16 tile plan,
 //    17 the tiles went to the tcgen05 kernel, 18 qkv partial sums (flat), 19 their width, 20 K ranges S,
-//    21 most tokens with a buffer per range, 22 cos_sin; f: 0 scale
+//    21 most tokens with a buffer per range, 22 cos_sin, 23 sinks (float32 [Hq], or 0); f: 0 scale, 1 soft cap of the scores (0: none)
 SB_EXPORT int sb_op_attention_tc(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   const SbTilePlan& plan = s->plan[op->i[16]];
@@ -580,7 +603,8 @@ SB_EXPORT int sb_op_attention_tc(const SbOp* op, const SbStep* s, void* stream) 
   const int tiles = op->i[17] ? 0 : plan.tiles;
   if (tiles <= 0 && plan.items <= 0) return SB_OP_SKIPPED;
   const int32_t* list = work(s, plan) + (op->i[17] ? 2 * plan.tiles : 0);
-  return sb_attention_tc(ptr<const void>(op->i[0]), ptr<void>(op->i[1]), ptr<const void>(op->i[2]), ptr<const int32_t>(op->i[3]),
-                         (int)op->i[4], (int)op->i[5], op->i[6], op->i[7], op->i[8], entry_meta(s), s->max_rows, list, tiles, plan.items,
-                         plan.chunks, scratch, ptr<int>(op->i[11]), Hq, Hkv, D, (int)op->i[15], static_cast<float>(op->f[0]), st);
+  return sb_attention_tc_extra(ptr<const void>(op->i[0]), ptr<void>(op->i[1]), ptr<const void>(op->i[2]), ptr<const int32_t>(op->i[3]),
+                               (int)op->i[4], (int)op->i[5], op->i[6], op->i[7], op->i[8], entry_meta(s), s->max_rows, list, tiles, plan.items,
+                               plan.chunks, scratch, ptr<int>(op->i[11]), Hq, Hkv, D, (int)op->i[15], static_cast<float>(op->f[0]),
+                               static_cast<float>(op->f[1]), ptr<const float>(op->i[23]), st);
 }

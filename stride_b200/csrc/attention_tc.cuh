@@ -38,6 +38,9 @@ struct AttnTcParams {
   int n_partials;
   int64_t partial_stride;
   const float* cos_sin;  // [positions][D / 2][2]
+  // kernels with EXTRA: capped scores and sinks (attention_math.cuh)
+  float cap_k;           // 0: no cap
+  const float* sinks;    // [Hq] float32, or null
 };
 
 // Row r of a tile is (position r / G, head r % G); G is not known at compile time, so the division is a multiplication.
@@ -203,11 +206,18 @@ __device__ __forceinline__ void pv_tile(float (*o)[4], const float (*s)[4], cons
 // (gid, gid + 8) and leaves their weights; m_t, l_t are the tile's maximum and sum per row. `full` (the same for the
 // whole warp): every row in use sees every key of the tile, so nothing is masked. kUpper = false: rows 8..15 are not
 // in use and are left out (maximum -inf, sum 0; their entries of s are not touched).
+// cap_k != 0: the scores are capped first.
 template <bool kUpper>
 __device__ __forceinline__ void tile_weights(float (*s)[4], float* m_t, float* l_t, int key0, const int* row_pos, const int* row_lo,
-                                             float c, int lane, bool full) {
+                                             float c, int lane, bool full, float cap_k = 0.0f) {
   constexpr int X = kUpper ? 4 : 2, H = kUpper ? 2 : 1;
   const int tq = lane & 3;
+  if (cap_k != 0.0f) {
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+      for (int x = 0; x < X; ++x) s[nt][x] = capped_score(s[nt][x], cap_k);
+  }
   if (!full) {
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt)
@@ -254,8 +264,9 @@ __device__ __forceinline__ void tile_weights(float (*s)[4], float* m_t, float* l
 // One tile for one warp: weights from the raw scores in s, then o_t = the tile's weighted values per row.
 template <int D, bool kUpper = true>
 __device__ __forceinline__ void tile_partial(float (*s)[4], float (*o_t)[4], float* m_t, float* l_t, int key0, const int* row_pos,
-                                             const int* row_lo, float c, const bf16* sV, int lane, bool full = false) {
-  tile_weights<kUpper>(s, m_t, l_t, key0, row_pos, row_lo, c, lane, full);
+                                             const int* row_lo, float c, const bf16* sV, int lane, bool full = false,
+                                             float cap_k = 0.0f) {
+  tile_weights<kUpper>(s, m_t, l_t, key0, row_pos, row_lo, c, lane, full, cap_k);
   pv_tile<D, kUpper>(o_t, s, sV, lane);
 }
 
@@ -327,25 +338,29 @@ __device__ __forceinline__ void fold_records(int c0, int c1, Load load, float& m
 }
 
 // The finished value of element (r, d) of one (entry, key/value head) from the records of its chunks c0..c1.
+// sink (or null): the row's sink.
 template <int D>
-__device__ __forceinline__ float fold_chunks(const float* part_o, const float* part_ml, int64_t rec0, int c0, int c1, int r, int d) {
+__device__ __forceinline__ float fold_chunks(const float* part_o, const float* part_ml, int64_t rec0, int c0, int c1, int r, int d,
+                                             const float* sink = nullptr) {
   float m = -INFINITY, l = 0.0f, o = 0.0f, unused = 0.0f;
   fold_records(c0, c1, [&](int c, float2& ml, float2& v) {
     ml = __ldcg(reinterpret_cast<const float2*>(&part_ml[((rec0 + c) * 16 + r) * 2]));
     v = make_float2(__ldcg(&part_o[(rec0 + c) * 16 * D + r * D + d]), 0.0f);
   }, m, l, o, unused);
+  if (sink != nullptr) l = with_sink(l, m, *sink);
   return finish(o, l);
 }
 
 // The same for elements (r, d) and (r, d + 1), d even: the row's factors are computed once.
 template <int D, bool AHEAD = true>
 __device__ __forceinline__ void fold_chunks2(const float* part_o, const float* part_ml, int64_t rec0, int c0, int c1, int r, int d,
-                                             float& a, float& b) {
+                                             float& a, float& b, const float* sink = nullptr) {
   float m = -INFINITY, l = 0.0f, o0 = 0.0f, o1 = 0.0f;
   fold_records<AHEAD>(c0, c1, [&](int c, float2& ml, float2& v) {
     ml = __ldcg(reinterpret_cast<const float2*>(&part_ml[((rec0 + c) * 16 + r) * 2]));
     v = __ldcg(reinterpret_cast<const float2*>(&part_o[(rec0 + c) * 16 * D + r * D + d]));
   }, m, l, o0, o1);
+  if (sink != nullptr) l = with_sink(l, m, *sink);
   a = finish(o0, l);
   b = finish(o1, l);
 }
@@ -404,7 +419,8 @@ __host__ __device__ constexpr size_t decode_unit_smem() {
 // record in global memory, a ticket and a second look at memory (3.2 us a layer for a decode step at the 1B sizes).
 template <int D>
 __host__ __device__ constexpr int decode_record_floats() { return 16 * (D + 2); }
-template <int D, bool FUSED, bool CLUSTER, class Env>
+// EXTRA: scores may be capped and rows may have sinks.
+template <int D, bool FUSED, bool CLUSTER, bool EXTRA, class Env>
 __device__ __forceinline__ void decode_unit(const AttnTcParams& p, int item, int g, int chunk, uint8_t* smem_tiles, int* is_last_p, int tid, Env& env,
                                             float* cluster_record = nullptr) {
   constexpr int LD = D + 8, CH = D / 8;
@@ -441,6 +457,7 @@ __device__ __forceinline__ void decode_unit(const AttnTcParams& p, int item, int
           v = sb::cluster_load_float2(sb::cluster_peer_address(cluster_record + r * D + d, c));
         }, m, l, o0, o1);
         const int pi = div_g(p, r);
+        if (EXTRA && p.sinks != nullptr) l = with_sink(l, m, p.sinks[g * G + r - pi * G]);
         *reinterpret_cast<uint32_t*>(p.out + (static_cast<int64_t>(first_row + pi) * p.Hq + g * G + r - pi * G) * D + d) =
             pack_bf16(finish(o0, l), finish(o1, l));
       }
@@ -527,8 +544,9 @@ __device__ __forceinline__ void decode_unit(const AttnTcParams& p, int item, int
       cp_commit();
     }
     const bool full = key0 + kKeys - 1 <= first_pos && key0 >= (p.window > 0 ? pos_hi - p.window + 1 : 0);
-    if (rows > 8) tile_weights<true>(s, m_t, l_t, key0, row_pos, row_lo, p.scale_log2, lane, full);
-    else tile_weights<false>(s, m_t, l_t, key0, row_pos, row_lo, p.scale_log2, lane, full);
+    const float cap_k = EXTRA ? p.cap_k : 0.0f;
+    if (rows > 8) tile_weights<true>(s, m_t, l_t, key0, row_pos, row_lo, p.scale_log2, lane, full, cap_k);
+    else tile_weights<false>(s, m_t, l_t, key0, row_pos, row_lo, p.scale_log2, lane, full, cap_k);
     if (!FUSED) {
       cp_wait<0>();
       __syncwarp();
@@ -583,6 +601,7 @@ __device__ __forceinline__ void decode_unit(const AttnTcParams& p, int item, int
         b = fold_value(b, o1, f);
       }
       const int pi = div_g(p, r);
+      if (EXTRA && p.sinks != nullptr) lr = with_sink(lr, m, p.sinks[g * G + r - pi * G]);
       *reinterpret_cast<uint32_t*>(p.out + (static_cast<int64_t>(first_row + pi) * p.Hq + g * G + r - pi * G) * D + d) =
           pack_bf16(finish(a, lr), finish(b, lr));
       continue;
@@ -615,8 +634,9 @@ __device__ __forceinline__ void decode_unit(const AttnTcParams& p, int item, int
   const int64_t rec0 = (static_cast<int64_t>(item) * p.Hkv + g) * p.chunks;
   for (int r = tid / PR; r < rows; r += 128 / PR) {
     float a, b;
-    fold_chunks2<D, Env::kFoldAhead>(p.part_o, p.part_ml, rec0, c0, c1, r, d, a, b);
     const int pi = div_g(p, r);
+    fold_chunks2<D, Env::kFoldAhead>(p.part_o, p.part_ml, rec0, c0, c1, r, d, a, b,
+                                     EXTRA && p.sinks != nullptr ? p.sinks + g * G + r - pi * G : nullptr);
     *reinterpret_cast<uint32_t*>(p.out + (static_cast<int64_t>(first_row + pi) * p.Hq + g * G + r - pi * G) * D + d) = pack_bf16(a, b);
   }
 }

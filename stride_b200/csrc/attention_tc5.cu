@@ -76,10 +76,13 @@ struct Fa5Params {
   const int32_t* work;                     // [tiles][2] = (entry, tile in entry)
   int Hq, Hkv, window;
   float scale_log2;
+  float cap_k;                             // EXTRA: capped scores (0: none) and sinks ([Hq] float32, or null), see attention_math.cuh
+  const float* sinks;
   int* status;
 };
 
-template <int D>
+// EXTRA: scores may be capped and rows may have sinks.
+template <int D, bool EXTRA>
 __global__ void __launch_bounds__(kThreads, 1)
 attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const Fa5Params p) {
   using SH = Shape<D>;
@@ -338,6 +341,10 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       tmem_load_wait();
       fence_before_sync();
       mbar_arrive(smem_u32(&s_free));      // this thread has its scores: the accumulator may be overwritten
+      if (EXTRA && p.cap_k != 0.0f) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j) sv[j] = __float_as_uint(capped_score(__uint_as_float(sv[j]), p.cap_k));
+      }
       if (span_masked(i)) {
         const int key0 = (kt0 + i) * kKeys + half * 64;
 #pragma unroll
@@ -433,6 +440,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     }
     fold_span(T - 1);
     if (valid) {
+      if (EXTRA && p.sinks != nullptr) l_r = with_sink(l_r, m_r, p.sinks[g * G + hh]);
       bf16* dst = p.out + (static_cast<int64_t>(row0 + pi) * p.Hq + g * G + hh) * D + half * kHalfD;
 #pragma unroll
       for (int c = 0; c < kHalfD / 8; ++c) {
@@ -466,11 +474,11 @@ SB_EXPORT int sb_attention_tc5_supported(int Hq, int Hkv, int D, int page_size) 
 
 // Attention of prompt portions. q, out: [n_tokens][Hq * D] bfloat16. k_base: this layer's keys of page 0 inside an
 // arena of `pages` pages; strides in elements. work: [n_tiles][2] = (entry, tile), a tile being 128 / (Hq / Hkv)
-// consecutive positions of the entry. meta as for sb_attention_tc.
-SB_EXPORT int sb_attention_tc5(const void* q, void* out, const void* k_base, int pages, const int32_t* block_table,
+// consecutive positions of the entry. meta as for sb_attention_tc. cap > 0: scores are capped softly; sinks: float32 [Hq], or null.
+SB_EXPORT int sb_attention_tc5_extra(const void* q, void* out, const void* k_base, int pages, const int32_t* block_table,
                                int max_pages, int page_size, int64_t page_stride, int64_t v_offset, int64_t head_stride,
                                const int32_t* meta, int meta_stride, const int32_t* work, int n_tiles, int n_tokens, int Hq,
-                               int Hkv, int D, int window, float scale, cudaStream_t stream) {
+                               int Hkv, int D, int window, float scale, float cap, const float* sinks, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (!sb_attention_tc5_supported(Hq, Hkv, D, page_size)) return sb::fail("sb_attention_tc5: shape not supported (Hq %d Hkv %d D %d page %d)", Hq, Hkv, D, page_size);
   if ((page_stride | v_offset | head_stride) % D != 0 || ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_base) | reinterpret_cast<uintptr_t>(out)) & 15))
@@ -496,7 +504,9 @@ SB_EXPORT int sb_attention_tc5(const void* q, void* out, const void* k_base, int
   p.Hq = Hq;
   p.Hkv = Hkv;
   p.window = window;
-  p.scale_log2 = scale * kLog2e;
+  p.scale_log2 = (cap > 0.0f ? cap : scale) * kLog2e;
+  p.cap_k = cap > 0.0f ? 2.0f * kLog2e * scale / cap : 0.0f;
+  p.sinks = sinks;
   p.status = status;
 
   CUtensorMap map_q, map_kv;
@@ -510,16 +520,33 @@ SB_EXPORT int sb_attention_tc5(const void* q, void* out, const void* k_base, int
     return sb::fail("sb_attention_tc5: cuTensorMapEncodeTiled failed");
   static sb::DeviceOnce once;
   if (once.needed()) {
-    if (cudaFuncSetAttribute(attn_prefill_tc5_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<64>::kSmemBytes + 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(attn_prefill_tc5_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<128>::kSmemBytes + 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(attn_prefill_tc5_kernel<64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<64>::kSmemBytes + 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(attn_prefill_tc5_kernel<64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<64>::kSmemBytes + 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(attn_prefill_tc5_kernel<128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<128>::kSmemBytes + 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(attn_prefill_tc5_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<128>::kSmemBytes + 1024) != cudaSuccess)
       return sb::fail("sb_attention_tc5: cannot raise the shared memory limit");
     once.done();
   }
-  if (D == 64)
-    sb::launch_pdl(attn_prefill_tc5_kernel<64>, dim3(n_tiles, Hkv), dim3(kThreads), static_cast<size_t>(Shape<64>::kSmemBytes + 1024), stream, map_q, map_kv, p);
-  else
-    sb::launch_pdl(attn_prefill_tc5_kernel<128>, dim3(n_tiles, Hkv), dim3(kThreads), static_cast<size_t>(Shape<128>::kSmemBytes + 1024), stream, map_q, map_kv, p);
+  const bool extra = cap > 0.0f || sinks != nullptr;
+#define SB_TC5(D_, X) \
+  sb::launch_pdl(attn_prefill_tc5_kernel<D_, X>, dim3(n_tiles, Hkv), dim3(kThreads), static_cast<size_t>(Shape<D_>::kSmemBytes + 1024), stream, map_q, map_kv, p)
+  if (D == 64) {
+    if (extra) SB_TC5(64, true);
+    else SB_TC5(64, false);
+  } else {
+    if (extra) SB_TC5(128, true);
+    else SB_TC5(128, false);
+  }
+#undef SB_TC5
   return sb::check_launch("sb_attention_tc5");
+}
+
+SB_EXPORT int sb_attention_tc5(const void* q, void* out, const void* k_base, int pages, const int32_t* block_table,
+                               int max_pages, int page_size, int64_t page_stride, int64_t v_offset, int64_t head_stride,
+                               const int32_t* meta, int meta_stride, const int32_t* work, int n_tiles, int n_tokens, int Hq,
+                               int Hkv, int D, int window, float scale, cudaStream_t stream) {
+  return sb_attention_tc5_extra(q, out, k_base, pages, block_table, max_pages, page_size, page_stride, v_offset, head_stride, meta, meta_stride,
+                                work, n_tiles, n_tokens, Hq, Hkv, D, window, scale, 0.0f, nullptr, stream);
 }
 
 // From now on the kernel reports into `device_word` (see sb_gemm_tc_use_status_word); null: into its own again.
@@ -538,13 +565,14 @@ SB_EXPORT int sb_attention_tc5_status() {
 // ------------------------------------------------------------------ operation of the native step program (step_ops.h)
 // The tiles of the step's tile plan (prompt portions) on the tcgen05 kernel.
 // i: 0 q, 1 out, 2 cache layer, 3 pages of the arena, 4 block table, 5 pages per sequence, 6 page size, 7 page stride,
-//    8 v offset, 9 head stride, 10 Hq, 11 Hkv, 12 D, 13 window, 14 tile plan; f: 0 scale
+//    8 v offset, 9 head stride, 10 Hq, 11 Hkv, 12 D, 13 window, 14 tile plan, 15 sinks (float32 [Hq], or 0); f: 0 scale, 1 soft cap of the scores (0: none)
 SB_EXPORT int sb_op_attention_tc5(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
   const SbTilePlan& plan = s->plan[op->i[14]];
   if (plan.fused || plan.tiles <= 0) return SB_OP_SKIPPED;
-  return sb_attention_tc5(ptr<const void>(op->i[0]), ptr<void>(op->i[1]), ptr<const void>(op->i[2]), (int)op->i[3],
+  return sb_attention_tc5_extra(ptr<const void>(op->i[0]), ptr<void>(op->i[1]), ptr<const void>(op->i[2]), (int)op->i[3],
                           ptr<const int32_t>(op->i[4]), (int)op->i[5], (int)op->i[6], op->i[7], op->i[8], op->i[9], entry_meta(s),
                           s->max_rows, work(s, plan), plan.tiles, s->n, (int)op->i[10], (int)op->i[11], (int)op->i[12], (int)op->i[13],
-                          static_cast<float>(op->f[0]), static_cast<cudaStream_t>(stream));
+                          static_cast<float>(op->f[0]), static_cast<float>(op->f[1]), ptr<const float>(op->i[15]),
+                          static_cast<cudaStream_t>(stream));
 }

@@ -34,7 +34,8 @@ typedef struct SbTilePlan {
   int32_t group, tile_rows, kv_heads, fused_limit;   // the key: what a mixer asked for
   int32_t work_offset, tiles, items, chunks;
   int32_t fused;        // the step has items only and few enough CTAs: rotation and append run inside the decode kernel
-  int32_t reserved[3];
+  int32_t reserved;
+  const int32_t* list;  // the list itself where it lies outside the step's integer inputs, else null
 } SbTilePlan;
 
 typedef struct SbStep {
@@ -67,7 +68,7 @@ inline const int32_t* positions(const SbStep* s) { return s->ints + s->max_rows;
 inline const int32_t* slots(const SbStep* s) { return s->ints + 2 * static_cast<int64_t>(s->max_rows); }
 inline const int32_t* wanted_rows(const SbStep* s) { return s->ints + 3 * static_cast<int64_t>(s->max_rows); }
 inline const int32_t* entry_meta(const SbStep* s) { return s->ints + 4 * static_cast<int64_t>(s->max_rows); }
-inline const int32_t* work(const SbStep* s, const SbTilePlan& p) { return s->ints + 9 * static_cast<int64_t>(s->max_rows) + p.work_offset; }
+inline const int32_t* work(const SbStep* s, const SbTilePlan& p) { return p.list != nullptr ? p.list : s->ints + 9 * static_cast<int64_t>(s->max_rows) + p.work_offset; }
 // Partial sums that a projection with K ranges left: [P, n, M] with P = S up to `few` tokens, else 1.
 inline int partial_count(int64_t S, int64_t few, int n) { return (S > 1 && n <= few) ? static_cast<int>(S) : 1; }
 template <class T>

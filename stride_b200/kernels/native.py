@@ -29,7 +29,7 @@ class NotNative(Exception):
 class SbTilePlan(ctypes.Structure):
     _fields_ = [("group", c_int32), ("tile_rows", c_int32), ("kv_heads", c_int32), ("fused_limit", c_int32),
                 ("work_offset", c_int32), ("tiles", c_int32), ("items", c_int32), ("chunks", c_int32),
-                ("fused", c_int32), ("reserved", c_int32 * 3)]
+                ("fused", c_int32), ("reserved", c_int32), ("list", c_void_p)]
 
 
 class SbStep(ctypes.Structure):
@@ -324,6 +324,31 @@ class ImmediateProgram(_StreamHolder):
         self.embedding_output = ctx.embedding_output
         self.pending = None
         self.chain = None
+        self._ctx, self._notes = ctx, []
+
+    def plan(self, group: int, tile_rows: int, kv_heads: int, fused_limit: int) -> int:
+        """The step's entries cut for the tensor-core attention kernels (no rotation inside the decode kernel)."""
+        if fused_limit >= 0:
+            raise NotNative("a step laid out at once has no fused plan")
+        step = self.step
+        for k in range(step.n_plans):
+            if (step.plan[k].group, step.plan[k].tile_rows) == (group, tile_rows):
+                return k
+        if step.n_plans >= MAX_PLANS:
+            raise NotNative(f"a part may ask for at most {MAX_PLANS} different tile plans")
+        work, tiles, items, chunks = self._ctx.tile_plan(group, tile_rows)
+        q = step.plan[step.n_plans]
+        q.group, q.tile_rows, q.kv_heads, q.fused_limit = group, tile_rows, kv_heads, fused_limit
+        q.tiles, q.items, q.chunks, q.fused, q.list = tiles, items, chunks, 0, work.data_ptr()
+        self._notes.append(work)
+        step.n_plans += 1
+        return step.n_plans - 1
+
+    def growing_buffer(self, name: str, dtype: torch.dtype, key, need) -> int:
+        buf = self.workspace.grow(name, need(self.step), dtype)
+        note = (c_int64 * 2)(buf.data_ptr(), buf.numel())
+        self._notes += [buf, note]
+        return ctypes.addressof(note)
 
     @property
     def streams(self):

@@ -23,6 +23,38 @@ from .base import CacheNeed, Mixer, part_class, register_part
 from .spec import TensorPlan
 
 
+def page_where(pages, table) -> list:
+    return [pages, table, table.shape[1], pages.shape[3], pages.stride(0), pages.stride(1), pages.stride(2)]
+
+
+def tensor_core_head(dtype, num_heads: int, num_kv_heads: int, head_dim: int) -> bool:
+    """True if the tensor-core attention kernels with heads of fixed size take this shape."""
+    return dtype == torch.bfloat16 and head_dim in (64, 128) and num_heads // num_kv_heads <= 16
+
+
+def emit_tensor_core_attention(program, q, out, pages, table, H: int, G: int, D: int, window: int, scale: float, plan: int, tc5: bool,
+                               projected=None, cap: float = 0.0, sinks=None) -> None:
+    """Prompt portions on the tcgen05 kernel where the page size allows it (`tc5`; else, and decoded tokens and very short portions always,
+    on the mma.sync kernels), each finding its share of the step in the step's tile plan. projected: (q | k | v partial sums, their width,
+    K ranges, rotation table) where the decode kernel may rotate and append itself. cap: scores are capped softly; sinks: a term exp(sink)
+    per head in the denominator."""
+    ws, where = program.workspace, page_where(pages, table)
+    if tc5:
+        program.add("attention_tc5", "sb_op_attention_tc5", [q, out, pages, pages.shape[0], *where[1:], H, G, D, window, plan, sinks], [scale, cap],
+                    chain=NO_PHASE)
+    # the decode kernel's chunk records: as many as the step's decode entries and their longest context need
+    need = ops.attention_tc_scratch
+    scratch = program.growing_buffer("attn.scratch", torch.float32, (plan, G, D), lambda step: need(step.plan[plan].items, G, step.plan[plan].chunks, D))
+    counters = ws.raw("attn.counters", (ws.max_tokens * G,), torch.int32)
+    qkv, width, S, cos_sin = projected or (None, 0, 1, None)
+    phase = None
+    if projected is not None:
+        phase = lambda chain: chain.attention(qkv, S, cos_sin, out, pages, table, scratch, counters, H, G, D, window, scale, plan)
+    program.add("attention_tc", "sb_op_attention_tc",
+                [q, out, *where, scratch, 0, counters, H, G, D, window, plan, int(tc5), qkv, width, S, program.few_tokens, cos_sin, sinks],
+                [scale, cap], chain=phase)
+
+
 @register_part("mixer", "attention")
 class AttentionMixer(Mixer):
     """params: hidden_size, num_heads, num_kv_heads, head_dim, window (0 = all keys),
@@ -91,34 +123,6 @@ class AttentionMixer(Mixer):
         return CacheNeed("pages", kv_heads=self.num_kv_heads, head_dim=self.head_dim, window=self.window,
                          dtype=self.env.act_dtype)
 
-    @staticmethod
-    def _tc_plan(ctx, G: int, tile_rows: int = 64):
-        """(work list on the device, tiles, items, chunks) of the tensor-core attention kernels for this
-        step: entries of at most 16 // G tokens go to the decode kernel (one item each), longer ones are
-        cut into tiles of tile_rows // G positions. Made once per step and shared by all layers of this ratio."""
-        key = ("attention_tc_plan", G, tile_rows)
-        plan = ctx.shared.get(key)
-        if plan is None and ctx.static_keys:
-            E = len(ctx.entry_length)
-            plan = (ctx.workspace.iota(E), 0, E, (ctx.static_keys + 255) // 256)
-            ctx.shared[key] = plan
-        if plan is None:
-            ppt, short = tile_rows // G, 16 // G
-            tiled, items, last = [], [], 0
-            for e, (L, p0) in enumerate(zip(ctx.entry_length, ctx.entry_first_pos)):
-                if L <= short:
-                    items.append(e)
-                    last = max(last, p0 + L - 1)
-                else:
-                    tiled += [(p0 + min(L, (t + 1) * ppt), e, t) for t in range((L + ppt - 1) // ppt)]
-            # the tiles that see the most keys first: CTAs start in this order, and the short ones fill the end
-            tiled.sort(key=lambda k: -k[0])
-            tiles = [x for _, e, t in tiled for x in (e, t)]
-            work = ctx.upload_ints(np.asarray(tiles + items, dtype=np.int32))
-            plan = (work, len(tiles) // 2, len(items), last // 256 + 1 if items else 0)
-            ctx.shared[key] = plan
-        return plan
-
     def kernel_libraries(self):
         if self.env.compute_dtype != torch.bfloat16:
             return {"gemm_f32", "elementwise", "attention_generic"}
@@ -132,11 +136,11 @@ class AttentionMixer(Mixer):
         qkv = self.qkv.forward_partials(x, ws.raw("attn.qkv", (self.qkv.partial_elems(ws.max_tokens),), torch.float32))
         mixed = ws.get("attn.out", n, (self.num_heads * D,), ctx.act_dtype)
         G = self.num_heads // self.num_kv_heads
-        tensor_core = ctx.act_dtype == torch.bfloat16 and D in (64, 128) and G <= 16
+        tensor_core = tensor_core_head(ctx.act_dtype, self.num_heads, self.num_kv_heads, D)
         plan = None
         if tensor_core:
             tc5 = ops.attention_tc5_supported(self.num_heads, self.num_kv_heads, D, cache.page_size)
-            plan = self._tc_plan(ctx, G, 128 if tc5 else 64)
+            plan = ctx.tile_plan(G, 128 if tc5 else 64)
         if (plan is not None and plan[1] == 0 and cache.writes and self._rotary == D and not self.values_from_keys
                 and plan[2] * self.num_kv_heads * plan[3] <= ops.attention_decode_rope_limit()):
             # only decoded tokens and very short portions, few enough for all CTAs to run at once: rotation and append
@@ -180,9 +184,9 @@ class AttentionMixer(Mixer):
         mixed = ws.get("attn.out", T, (self.num_heads * D,), act)
         q = ws.get("attn.q", T, (self.num_heads * D,), act)
         G = self.num_heads // self.num_kv_heads
-        tensor_core = act == torch.bfloat16 and D in (64, 128) and G <= 16
+        tensor_core = tensor_core_head(act, self.num_heads, self.num_kv_heads, D)
         pages, table = cache.pages, cache.block_table
-        where = [pages, table, table.shape[1], pages.shape[3], pages.stride(0), pages.stride(1), pages.stride(2)]
+        where = page_where(pages, table)
         plan = -1
         if tensor_core:
             tc5 = ops.attention_tc5_supported(self.num_heads, self.num_kv_heads, D, cache.page_size)
@@ -196,20 +200,8 @@ class AttentionMixer(Mixer):
                      self.num_kv_heads, D, int(cache.writes), plan, int(self.values_from_keys)],
                     chain=NO_PHASE if tensor_core and fused else None)
         if tensor_core:
-            if tc5:
-                program.add("attention_tc5", "sb_op_attention_tc5",
-                            [q, mixed, pages, pages.shape[0], *where[1:], self.num_heads, self.num_kv_heads, D, self.window, plan], [self.scale],
-                            chain=NO_PHASE)
-            # the decode kernel's chunk records: as many as the step's decode entries and their longest context need
-            kv, need = self.num_kv_heads, ops.attention_tc_scratch
-            scratch = program.growing_buffer("attn.scratch", torch.float32, (plan, kv, D),
-                                             lambda step, k=plan: need(step.plan[k].items, kv, step.plan[k].chunks, D))
-            counters = ws.raw("attn.counters", (T * self.num_kv_heads,), torch.int32)
-            program.add("attention_tc", "sb_op_attention_tc",
-                        [q, mixed, *where, scratch, 0, counters, self.num_heads, self.num_kv_heads, D, self.window, plan,
-                         int(tc5), qkv, self.qkv_width, S, program.few_tokens, self._cos_sin], [self.scale],
-                        chain=lambda chain: chain.attention(qkv, S, self._cos_sin, mixed, pages, table, scratch, counters, self.num_heads,
-                                                            self.num_kv_heads, D, self.window, self.scale, plan))
+            emit_tensor_core_attention(program, q, mixed, pages, table, self.num_heads, self.num_kv_heads, D, self.window, self.scale, plan, tc5,
+                                       projected=(qkv, self.qkv_width, S, self._cos_sin))
         else:
             program.add("attention_generic", "sb_op_attention_generic",
                         [q, mixed, q.dtype, *where, self.num_heads, self.num_kv_heads, D, self.window], [self.scale])

@@ -5,6 +5,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Optional
 
+import numpy as np
 import torch
 
 
@@ -121,6 +122,33 @@ class StepContext:
     def act_dtype(self) -> torch.dtype:
         return self.compute_dtype
 
+    def tile_plan(self, group: int, tile_rows: int = 64):
+        """(work list on the device, tiles, items, chunks) of the tensor-core attention kernels for this
+        step: entries of at most 16 // group tokens go to the decode kernel (one item each), longer ones are
+        cut into tiles of tile_rows // group positions. Made once per step and shared by all layers of this ratio."""
+        key = ("attention_tc_plan", group, tile_rows)
+        plan = self.shared.get(key)
+        if plan is None and self.static_keys:
+            E = len(self.entry_length)
+            plan = (self.workspace.iota(E), 0, E, (self.static_keys + 255) // 256)
+            self.shared[key] = plan
+        if plan is None:
+            ppt, short = tile_rows // group, 16 // group
+            tiled, items, last = [], [], 0
+            for e, (L, p0) in enumerate(zip(self.entry_length, self.entry_first_pos)):
+                if L <= short:
+                    items.append(e)
+                    last = max(last, p0 + L - 1)
+                else:
+                    tiled += [(p0 + min(L, (t + 1) * ppt), e, t) for t in range((L + ppt - 1) // ppt)]
+            # the tiles that see the most keys first: CTAs start in this order, and the short ones fill the end
+            tiled.sort(key=lambda k: -k[0])
+            tiles = [x for _, e, t in tiled for x in (e, t)]
+            work = self.upload_ints(np.asarray(tiles + items, dtype=np.int32))
+            plan = (work, len(tiles) // 2, len(items), last // 256 + 1 if items else 0)
+            self.shared[key] = plan
+        return plan
+
     @property
     def decode_only(self) -> bool:
         return all(l == 1 for l in self.entry_length)
@@ -146,4 +174,5 @@ def step_context(entries, workspace: Workspace, compute_dtype: torch.dtype, toke
     E = len(entries)
     return StepContext(n=n, token_ids=d[0:n], positions=d[R:R + n], slots=d[2 * R:2 * R + n], workspace=workspace, compute_dtype=compute_dtype,
                        entry_slots=[e[0] for e in entries], entry_first_row=[int(ints[5 * R + k]) for k in range(E)],
-                       entry_length=[e[1] for e in entries], entry_first_pos=[e[2] for e in entries], entry_meta=d[4 * R:8 * R].view(4, R)[:, :E])
+                       entry_length=[e[1] for e in entries], entry_first_pos=[e[2] for e in entries], entry_meta=d[4 * R:8 * R].view(4, R)[:, :E],
+                       upload_ints=lambda values: torch.from_numpy(np.ascontiguousarray(values, dtype=np.int32)).to(workspace.device))

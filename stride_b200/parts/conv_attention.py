@@ -1,5 +1,5 @@
-"""Softmax attention over the paged cache whose q, k and v pass a short causal convolution over time (kernels: csrc/short_conv.cu in front,
-csrc/masked_attention.cu).
+"""Softmax attention over the paged cache whose q, k and v pass a short causal convolution over time (kernels: csrc/short_conv.cu in front;
+csrc/attention_tc5.cu and attention_tc.cu for heads of 64 or 128 in the bfloat16 engine, csrc/masked_attention.cu otherwise).
 
 q, k, v = W x, no biases; each channel of them convolved over the last `taps` tokens (the last tap the current token's, zeros before the
 start). The first `rotary_dim` elements of every q and k head may be rotated by the position, and every head of them may then be divided by
@@ -18,6 +18,7 @@ from ..kernels import ops
 from ..kernels.linear import Linear
 from ..kernels.native import ImmediateProgram
 from .base import CacheNeed, Mixer, part_class, register_part
+from .attention import emit_tensor_core_attention, tensor_core_head
 from .masked_attention import _emit_attend, _page_where
 from .spec import TensorPlan
 
@@ -101,7 +102,11 @@ class ConvAttentionMixer(Mixer):
         return [pages, CacheNeed("state", state_shape=(self.record,), state_dtype=torch.float32)]
 
     def kernel_libraries(self):
-        return {"short_conv", "masked_attention", "gemm_tc" if self.env.compute_dtype == torch.bfloat16 else "gemm_f32"}
+        attend = {"attention_tc", "attention_tc5"} if self._fixed_heads() else {"masked_attention"}
+        return attend | {"short_conv", "gemm_tc" if self.env.compute_dtype == torch.bfloat16 else "gemm_f32"}
+
+    def _fixed_heads(self) -> bool:
+        return self.D == self.V and tensor_core_head(self.env.act_dtype, self.H, self.G, self.D)
 
     def _tiles(self, pages) -> bool:
         return self.env.act_dtype == torch.bfloat16 and ops.masked_attention_tiles_supported(self.H, self.G, self.D, self.V, pages.shape[4],
@@ -125,5 +130,10 @@ class ConvAttentionMixer(Mixer):
                     [qkv, self.channels, S, program.few_tokens, self.conv, self.taps, state, self.record, self.cos_sin, self.rot, int(self.unit), kept,
                      {None: 0, "keep": 1, "mix": 2}[self.value_mix], q, q.dtype, pages, table, *_page_where(pages, table), H, G, D, V, pages.shape[4]],
                     [self.eps, self.lam])
-        _emit_attend(program, q, mixed, paged, None, self.sinks, H, G, D, V, self.window, 0, self.scale, self._tiles(pages), cap=self.cap)
+        if self._fixed_heads():
+            tc5 = ops.attention_tc5_supported(H, G, D, pages.shape[3])
+            plan = program.plan(H // G, 128 if tc5 else 64, 1, -1)
+            emit_tensor_core_attention(program, q, mixed, pages, table, H, G, D, self.window, self.scale, plan, tc5, cap=self.cap, sinks=self.sinks)
+        else:
+            _emit_attend(program, q, mixed, paged, None, self.sinks, H, G, D, V, self.window, 0, self.scale, self._tiles(pages), cap=self.cap)
         self.o.emit_add(program, mixed, ws.raw("cattn.o_partials", (self.o.partial_elems(T),), f32))
