@@ -1121,12 +1121,12 @@ def _mezadra_kernels(timed, pk: dict, width: int, ff: int) -> dict:
         # between two sublayers: the norm on a result with the second output; Keralorn's layer norm in front of one
         P = 1 if n > 512 else 8
         h, parts, two, x = rand(n, width), rand(P, n, width), rand(n, width), torch.empty(n, width, dtype=bf, device=dev)
-        fold = lambda b, factor: op("branch", "sb_op_branch_norm_fold", [h, None, parts, P, 512, b, None, 1, gain, f32, width, 0, 0, None, factor, x], [1.0, 1.0, 1e-5])
+        fold = lambda b, factor: op("branch", "sb_op_branch_norm_fold", [h, None, parts, P, 512, None, b, 1, gain, f32, width, 0, 0, None, factor, x, 1], [1.0, 1.0, 1e-5])
         ms = timed(fold(None, None), 5, clear=True)
         record("norm_fold_" + label, ms, n * width * (10.0 + 4.0 * P))
         factor = rand(n)
         ms = timed(fold(two, factor), 5, clear=True)
-        record("norm_fold_two_sources_" + label, ms, n * width * (18.0 + 4.0 * P))
+        record("norm_fold_two_sources_" + label, ms, n * width * (14.0 + 4.0 * P))
         bias = torch.zeros(width, device=dev)
         ms = timed(lambda: ops.layernorm(h, gain, bias, 1e-5, x, partials=parts), 5, clear=True)
         record("keralorn_layernorm_" + label, ms, n * width * (10.0 + 4.0 * P))

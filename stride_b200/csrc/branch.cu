@@ -35,6 +35,7 @@ struct Source {
   int64_t stride;
   float c;
   const float* row_factor = nullptr;      // [n]: times c, or null
+  bool clear = true;                      // the buffer is zero afterwards
 };
 __device__ __forceinline__ float factor(const Source& s) {       // (a block is a row)
   return s.row_factor != nullptr ? __fmul_rn(s.c, s.row_factor[blockIdx.x]) : s.c;
@@ -47,7 +48,7 @@ __device__ __forceinline__ void narrow4(bf16* dst, float4 v) {
   *reinterpret_cast<uint2*>(dst) = packed;
 }
 
-// One element of a branch: its buffer (zero behind the read) plus its partial sums, h + (p0 + p1 + ..).
+// One element of a branch: its buffer (CLEAR: zero behind the read, if the branch wants it) plus its partial sums, h + (p0 + p1 + ..).
 template <class V>
 __device__ __forceinline__ V zero_of();
 template <>
@@ -60,13 +61,13 @@ __device__ __forceinline__ float mul(float a, float c) { return __fmul_rn(a, c);
 __device__ __forceinline__ float4 mul(float4 a, float c) { return make_float4(__fmul_rn(a.x, c), __fmul_rn(a.y, c), __fmul_rn(a.z, c), __fmul_rn(a.w, c)); }
 __device__ __forceinline__ float4 mul(float4 a, float4 c) { return make_float4(__fmul_rn(a.x, c.x), __fmul_rn(a.y, c.y), __fmul_rn(a.z, c.z), __fmul_rn(a.w, c.w)); }
 
-template <class V>
+template <class V, bool CLEAR = true>
 __device__ __forceinline__ V source_value(const Source& s, int64_t i) {      // i in units of V
   V v = zero_of<V>();
   if (s.h != nullptr) {
     V* h = reinterpret_cast<V*>(s.h) + i;
     v = *h;
-    *h = zero_of<V>();
+    if (CLEAR && s.clear) *h = zero_of<V>();
   }
   if (s.partials != nullptr && s.n_partials > 0) {
     const V* p = reinterpret_cast<const V*>(s.partials) + i;
@@ -83,6 +84,11 @@ __device__ __forceinline__ V source_value(const Source& s, int64_t i) {      // 
     v = s.h != nullptr ? add(v, sum) : sum;
   }
   return v;
+}
+
+template <class V>
+__device__ __forceinline__ void source_clear(const Source& s, int64_t i) {
+  if (s.h != nullptr && s.clear) reinterpret_cast<V*>(s.h)[i] = zero_of<V>();
 }
 
 template <class TG>
@@ -144,8 +150,8 @@ __global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict
     float4* held = reinterpret_cast<float4*>(row_values);
     for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
       const int64_t i = (row + c) / 4;
-      float4 v = mul(source_value<float4>(a, i), ca);
-      if (two) v = add(v, mul(source_value<float4>(b, i), cb));
+      float4 v = mul(source_value<float4, false>(a, i), ca);       // (cleared below: a store here would hold up the next requests)
+      if (two) v = add(v, mul(source_value<float4, false>(b, i), cb));
       held[c / 4] = v;
       sq = fmaf(v.x, v.x, sq), sq = fmaf(v.y, v.y, sq), sq = fmaf(v.z, v.z, sq), sq = fmaf(v.w, v.w, sq);
     }
@@ -157,6 +163,8 @@ __global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict
       v = add(*d, v);
       *d = v;
       if (copy != nullptr) narrow4(copy + row + c, v);
+      source_clear<float4>(a, (row + c) / 4);
+      source_clear<float4>(b, (row + c) / 4);
     }
     return;
   }
@@ -209,10 +217,10 @@ inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 }  // namespace
 
 SB_EXPORT int sb_branch_fold_ex(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, const float* ra, float* b, const float* pb, int nb,
-                                int64_t sb_, float cb, const float* rb, const void* gain, int gain_dtype, int n, int W, cudaStream_t stream) {
+                                int64_t sb_, float cb, const float* rb, int clear, const void* gain, int gain_dtype, int n, int W, cudaStream_t stream) {
   if (n <= 0 || W <= 0) return 0;
   if (a == nullptr && pa == nullptr) return sb::fail("sb_branch_fold: the first branch has neither a buffer nor partial sums");
-  const Source A{a, pa, pa ? na : 0, sa, ca, ra}, B{b, pb, pb ? nb : 0, sb_, cb, rb};
+  const Source A{a, pa, pa ? na : 0, sa, ca, ra, clear != 0}, B{b, pb, pb ? nb : 0, sb_, cb, rb, clear != 0};
   const bool vec = W % 4 == 0 && aligned16(dst) && aligned16(a) && aligned16(pa) && aligned16(b) && aligned16(pb) && aligned16(gain) &&
                    sa % 4 == 0 && sb_ % 4 == 0;
   const int threads = W >= 1024 ? 256 : 128;
@@ -232,16 +240,16 @@ SB_EXPORT int sb_branch_fold_ex(float* dst, float* a, const float* pa, int na, i
 
 SB_EXPORT int sb_branch_fold(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, float* b, const float* pb, int nb, int64_t sb_,
                              float cb, const void* gain, int gain_dtype, int n, int W, cudaStream_t stream) {
-  return sb_branch_fold_ex(dst, a, pa, na, sa, ca, nullptr, b, pb, nb, sb_, cb, nullptr, gain, gain_dtype, n, W, stream);
+  return sb_branch_fold_ex(dst, a, pa, na, sa, ca, nullptr, b, pb, nb, sb_, cb, nullptr, 1, gain, gain_dtype, n, W, stream);
 }
 
-// ra, rb [n]: a factor per row on each branch, or null. copy: the new rows as bfloat16, or null.
+// ra, rb [n]: a factor per row on each branch, or null. clear: the branches' buffers are zero afterwards. copy: the new rows as bfloat16, or null.
 SB_EXPORT int sb_branch_norm_fold_ex(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, const float* ra, float* b, const float* pb,
-                                     int nb, int64_t sb_, float cb, const float* rb, const void* gain, int gain_dtype, float eps, void* copy, int n,
+                                     int nb, int64_t sb_, float cb, const float* rb, int clear, const void* gain, int gain_dtype, float eps, void* copy, int n,
                                      int W, cudaStream_t stream) {
   if (n <= 0 || W <= 0) return 0;
   if (a == nullptr && pa == nullptr) return sb::fail("sb_branch_norm_fold: the first branch has neither a buffer nor partial sums");
-  const Source A{a, pa, pa ? na : 0, sa, ca, ra}, B{b, pb, pb ? nb : 0, sb_, cb, rb};
+  const Source A{a, pa, pa ? na : 0, sa, ca, ra, clear != 0}, B{b, pb, pb ? nb : 0, sb_, cb, rb, clear != 0};
   const size_t smem = static_cast<size_t>(W) * sizeof(float);
   if (smem > 160 * 1024) return sb::fail("sb_branch_norm_fold: a row of %d elements does not fit the row buffer", W);
   const bool vec = W % 4 == 0 && aligned16(dst) && aligned16(a) && aligned16(pa) && aligned16(b) && aligned16(pb) && aligned16(gain) &&
@@ -268,7 +276,7 @@ SB_EXPORT int sb_branch_norm_fold_ex(float* dst, float* a, const float* pa, int 
 
 SB_EXPORT int sb_branch_norm_fold(float* dst, float* a, const float* pa, int na, int64_t sa, float ca, float* b, const float* pb, int nb,
                                   int64_t sb_, float cb, const void* gain, int gain_dtype, float eps, int n, int W, cudaStream_t stream) {
-  return sb_branch_norm_fold_ex(dst, a, pa, na, sa, ca, nullptr, b, pb, nb, sb_, cb, nullptr, gain, gain_dtype, eps, nullptr, n, W, stream);
+  return sb_branch_norm_fold_ex(dst, a, pa, na, sa, ca, nullptr, b, pb, nb, sb_, cb, nullptr, 1, gain, gain_dtype, eps, nullptr, n, W, stream);
 }
 
 SB_EXPORT int sb_stream_add(float* dst, const float* partials, int n_partials, int64_t stride, const float* other, const void* vector,
@@ -297,7 +305,8 @@ SB_EXPORT int sb_row_scaled_add(float* dst, const void* x, int x_dtype, const fl
 
 // ------------------------------------------------------------------ operations of the native step program (step_ops.h)
 // i: 0 dst, 1 a, 2 a's partial sums (flat), 3 their K ranges S, 4 most tokens with a buffer per range, 5 b, 6 b's partial sums, 7 their S,
-//    8 gain, 9 gain dtype, 10 W, 11 a limit of a's own in place of i[4] (or 0), 12 the same for b, 13 a factor per row on a (or 0), 14 on b
+//    8 gain, 9 gain dtype, 10 W, 11 a limit of a's own in place of i[4] (or 0), 12 the same for b, 13 a factor per row on a (or 0), 14 on b,
+//    16 the branches' buffers need not be cleared
 // f: 0 ca, 1 cb
 SB_EXPORT int sb_op_branch_fold(const SbOp* op, const SbStep* s, void* stream) {
   using namespace sbstep;
@@ -307,7 +316,7 @@ SB_EXPORT int sb_op_branch_fold(const SbOp* op, const SbStep* s, void* stream) {
   return sb_branch_fold_ex(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
                         static_cast<float>(op->f[0]), ptr<const float>(op->i[13]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]),
                         partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n), stride, static_cast<float>(op->f[1]), ptr<const float>(op->i[14]),
-                        ptr<const void>(op->i[8]), (int)op->i[9], s->n, W, static_cast<cudaStream_t>(stream));
+                        op->i[16] == 0, ptr<const void>(op->i[8]), (int)op->i[9], s->n, W, static_cast<cudaStream_t>(stream));
 }
 
 // i: as sb_op_branch_fold, 15 the new rows once more as bfloat16 (or 0)      f: 0 ca, 1 cb, 2 eps
@@ -319,7 +328,7 @@ SB_EXPORT int sb_op_branch_norm_fold(const SbOp* op, const SbStep* s, void* stre
   return sb_branch_norm_fold_ex(ptr<float>(op->i[0]), ptr<float>(op->i[1]), ptr<const float>(op->i[2]), partial_count(op->i[3], op->i[11] ? op->i[11] : op->i[4], s->n), stride,
                              static_cast<float>(op->f[0]), ptr<const float>(op->i[13]), ptr<float>(op->i[5]), ptr<const float>(op->i[6]),
                              partial_count(op->i[7], op->i[12] ? op->i[12] : op->i[4], s->n), stride, static_cast<float>(op->f[1]),
-                             ptr<const float>(op->i[14]), ptr<const void>(op->i[8]), (int)op->i[9], static_cast<float>(op->f[2]), ptr<void>(op->i[15]),
+                             ptr<const float>(op->i[14]), op->i[16] == 0, ptr<const void>(op->i[8]), (int)op->i[9], static_cast<float>(op->f[2]), ptr<void>(op->i[15]),
                              s->n, W, static_cast<cudaStream_t>(stream));
 }
 

@@ -105,11 +105,11 @@ __device__ __forceinline__ void store_tile(uint32_t tmem_row, float* out, int m,
 // The SwiGLU epilogue of one accumulator tile by the four epilogue warps (128 threads that meet on named barrier 1):
 // lanes 0..63 of the tile hold 64 gate rows, lanes 64..127 the matching up rows; out[n, j] = silu(gate) * up as
 // bfloat16, j = tile_m * 64 + row. `quarter` = warp % 4 (the TMEM lanes this warp may read), xch: 16 x 64 floats of
-// shared memory that nothing else uses meanwhile. pair_weight (or null): column n stands for pair order[n], whose input is multiplied by
-// pair_weight[order[n]]; both products are linear in it, so the accumulators are.
+// shared memory that nothing else uses meanwhile. column_weight (or null; in shared memory): a factor on the
+// input of every column of the tile; both products are linear in it, so the accumulators are multiplied.
 __device__ __forceinline__ void swiglu_tile(uint32_t tmem_base, float* xch, bf16* out, int64_t ldo, int tile_m, int half_rows, int n0,
                                             int N, int BN, int quarter, int lane, bool ok, const Gate& gate = Gate(),
-                                            const float* pair_weight = nullptr, const int32_t* order = nullptr) {
+                                            const float* column_weight = nullptr) {
   const int j = tile_m * 64 + (quarter & 1) * 32 + lane;  // output feature
   for (int c0 = 0; c0 < BN; c0 += 16) {
     float v[16];
@@ -131,10 +131,7 @@ __device__ __forceinline__ void swiglu_tile(uint32_t tmem_base, float* xch, bf16
         if (n < N) {
           const float other = xch[(cb + c) * 64 + (quarter & 1) * 32 + lane];
           float g = quarter >= 2 ? other : v[c], u = quarter >= 2 ? v[8 + c] : other;
-          if (pair_weight != nullptr) {
-            const float w = pair_weight[order[n]];
-            g *= w, u *= w;
-          }
+          if (column_weight != nullptr) g *= column_weight[c0 + cb + c], u *= column_weight[c0 + cb + c];
           out[static_cast<int64_t>(n) * ldo + j] = __float2bfloat16_rn(gated_product(g, u, gate));
         }
       }

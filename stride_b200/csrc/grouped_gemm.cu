@@ -147,6 +147,7 @@ grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
   __shared__ __align__(8) uint64_t empty_bar[kMaxStages];
   __shared__ __align__(8) uint64_t accum_bar;
   __shared__ uint32_t tmem_base_s;
+  __shared__ float column_weight[EPI == kSwiglu ? 128 : 1];
 
   sb::grid_launch_dependents();
   sb::grid_dependency_wait();                    // which expert this tile belongs to is the sort's result
@@ -160,6 +161,10 @@ grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
   const int tile_m = blockIdx.x, iters = (p.K + kTileK - 1) / kTileK;
   const uint32_t tmem_cols = tmem_alloc_cols(BN);
 
+  if (EPI == kSwiglu && p.pair_weight != nullptr && threadIdx.x >= 64) {       // (the epilogue's warps: a tile has at most 128 rows)
+    const int n = n0 + threadIdx.x - 64;
+    column_weight[threadIdx.x - 64] = n < end ? p.pair_weight[p.order[n]] : 0.0f;
+  }
   if (threadIdx.x == 0) {
     prefetch_tensormap(&map_w);
     prefetch_tensormap(&map_x);
@@ -223,7 +228,7 @@ grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
     if (EPI == kSwiglu) {
       float* xch = reinterpret_cast<float*>(smem_raw + (smem0 - smem_u32(smem_raw)));      // stage 0 is free by now
       swiglu_tile(tmem_base, xch, static_cast<bf16*>(p.out), p.half_rows, tile_m, p.half_rows, n0, end, BN, quarter, lane, ok,
-                  Gate(), p.pair_weight, p.order);
+                  Gate(), p.pair_weight != nullptr ? column_weight : nullptr);
     } else {
       const int m = tile_m * kTileM + quarter * 32 + lane;
       for (int c0 = 0; c0 < BN && n0 + c0 < end; c0 += 16) {

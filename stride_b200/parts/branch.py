@@ -88,10 +88,12 @@ class LayerScale(BranchScale):
         (b, pb), cb = (sources[1][0].source(), sources[1][1]) if len(sources) > 1 else ((None, None), 1.0)
         ops.branch_fold(stream.h, a=a, a_partials=pa, ca=ca, b=b, b_partials=pb, cb=cb, gain=self.weight)
 
-    def emit(self, program, sources):
-        """sources: one or two (buffer or None, pending partial sums or None, constant)."""
+    def emit(self, program, sources, copy=None, fresh: bool = False):
+        """sources: one or two (buffer or None, pending partial sums or None, constant); copy, fresh: see BranchRMSNorm."""
         program.need_folded("a layer scale")
-        emit_fold(program, sources, self.weight, self.size)
+        emit_fold(program, sources, self.weight, self.size, fresh=fresh)
+        if copy is not None:
+            program.add("elementwise", "sb_op_cast_columns", [program.h, self.size, 1, program.few_tokens, 0, self.size, copy, copy.dtype])
 
 
 @register_part("branch_scale", "rmsnorm")
@@ -127,10 +129,11 @@ class BranchRMSNorm(BranchScale):
         (b, pb), cb = (sources[1][0].source(), sources[1][1]) if len(sources) > 1 else ((None, None), 1.0)
         ops.branch_norm_fold(stream.h, self.weight, self.eps, a=a, a_partials=pa, ca=ca, b=b, b_partials=pb, cb=cb)
 
-    def emit(self, program, sources, copy=None):
-        """`copy`: a bfloat16 buffer that the stream's new rows are stored in once more, for a sublayer that reads the stream itself."""
+    def emit(self, program, sources, copy=None, fresh: bool = False):
+        """`copy`: a bfloat16 buffer that the stream's new rows are stored in once more, for a sublayer that reads the stream itself.
+        `fresh`: the branches' buffers need not be zero afterwards."""
         program.need_folded("a norm behind a sublayer")
-        emit_fold(program, sources, self.weight, self.size, norm_eps=self.eps, copy=copy)
+        emit_fold(program, sources, self.weight, self.size, norm_eps=self.eps, copy=copy, fresh=fresh)
 
 
 ALWAYS = 1 << 30      # the limit of partial sums that are never added by the kernel that makes them, however many tokens a step has
@@ -141,10 +144,10 @@ def pending_limit(pending) -> int:
     return pending[3] if pending is not None and len(pending) > 3 else 0
 
 
-def emit_fold(program, sources, gain, width: int, norm_eps: float = None, copy=None) -> None:
+def emit_fold(program, sources, gain, width: int, norm_eps: float = None, copy=None, fresh: bool = False) -> None:
     """The operation that takes one or two branches (buffer or None, pending or None, constant) into the program's stream; with
     `norm_eps` their sum is RMS-normed over its row before the gain (and the new rows may go to a bfloat16 `copy` too). A branch's constant
-    may be a float32 tensor instead: a factor per row."""
+    may be a float32 tensor instead: a factor per row. `fresh`: the branches' buffers are not set back to zero (whoever fills them next stores)."""
     if not 1 <= len(sources) <= 2:
         raise ValueError("a fold takes one or two branches")
     (a, pa, ca), (b, pb, cb) = sources[0], sources[1] if len(sources) > 1 else (None, None, 1.0)
@@ -152,12 +155,12 @@ def emit_fold(program, sources, gain, width: int, norm_eps: float = None, copy=N
     if a is None and fa is None:
         raise ValueError("a branch that nothing wrote into")
     ints = [program.h, a, fa, Sa, program.few_tokens, b, fb, Sb, gain, gain.dtype if gain is not None else 0, width,
-            pending_limit(pa), pending_limit(pb), *(c if isinstance(c, torch.Tensor) else None for c in (ca, cb))]
+            pending_limit(pa), pending_limit(pb), *(c if isinstance(c, torch.Tensor) else None for c in (ca, cb)), copy, int(fresh)]
     ca, cb = (1.0 if isinstance(c, torch.Tensor) else c for c in (ca, cb))
     if norm_eps is None:
         program.add("branch", "sb_op_branch_fold", ints, [ca, cb])
     else:       # the branches' sum is RMS-normed over its row on the way
-        program.add("branch", "sb_op_branch_norm_fold", [*ints, copy], [ca, cb, norm_eps])
+        program.add("branch", "sb_op_branch_norm_fold", ints, [ca, cb, norm_eps])
 
 
 class _ScaledBlock(Block):
@@ -253,7 +256,7 @@ class _PostNormBlock(Block):
         copy = None
         if self.env.act_dtype != torch.float32:
             copy = ws.get("block.x", ws.max_tokens, (program.h.shape[1],), self.env.act_dtype)
-        scale.emit(program, sources, copy)
+        scale.emit(program, sources, copy, fresh=True)
         if copy is not None:
             program.note_narrow(copy)
 

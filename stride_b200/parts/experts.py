@@ -227,7 +227,7 @@ class GroupedExpertsFeedForward(FeedForward):
 
     def emit(self, program, x):
         program.need_folded("grouped experts")
-        emit_fold(program, self.emit_sources(program, x), None, self.hidden)
+        emit_fold(program, self.emit_sources(program, x), None, self.hidden, fresh=True)
 
     def _emit_grouped(self, program, x, choice, vocab: int, pair_weight, scale: float) -> list:
         """The chosen experts' and the shared expert's results as branches with constants. choice [vocab, top]: the experts of every token

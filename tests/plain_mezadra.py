@@ -35,7 +35,7 @@ def silu(z):
 
 def embed(tensors, cfg, tokens):
     """[T, W]: the tokens' rows of the table, scaled."""
-    return w(tensors, "embed")[torch.as_tensor(tokens)] * cfg["embedding"]["scale"]
+    return w(tensors, "embed")[torch.as_tensor(tokens)] * cfg.get("embedding", {}).get("scale", 1.0)
 
 
 def short_conv(u, taps):

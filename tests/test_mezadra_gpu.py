@@ -246,7 +246,7 @@ def test_one_key_that_stands_out_is_never_out_of_sight(dtype, D):
     from stride_b200.parts import ResidualStream, Workspace
     g = torch.Generator().manual_seed(9)
     H, G, V, W, page, n, loud = 4, 2, D, 64, 16, 330, 21
-    m = {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": 16.0 / D, "softcap": 9.0}
+    m = {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": 16.0 / D, "softcap": 5.0}
     t = _attention_case(H, G, D, V, W, 0, g, mixes=False)
     t["p.q"], t["p.k"] = torch.zeros(H * D, W, dtype=BF), torch.zeros(G * D, W, dtype=BF)
     for a in range(H):                                                  # every query points along its first element ..
@@ -274,7 +274,7 @@ def test_one_key_that_stands_out_is_never_out_of_sight(dtype, D):
     without = h.clone()
     without[loud, 1], without[loud, 2] = 0.0, 1.0
     for other in (plain.attention(without.double(), t, "p.", m, 1e-6, None, rnd)[0], plain.attention(h.double(), t, "p.", {**m, "softcap": 0.0}, 1e-6, None, rnd)[0]):
-        assert float((other - want)[loud + 1:].abs().max(dim=1).values.min()) > 0.15 * float(want.abs().max())
+        assert float((other - want)[loud + 1:].abs().max(dim=1).values.min()) > 0.04 * float(want.abs().max())
 
 
 @pytest.mark.parametrize("n,W,ff,dtype", [(5, 40, 24, torch.float32), (64, 100, 37, BF), (16, 64, 40, BF), (200, 128, 200, BF), (700, 256, 512, BF),
