@@ -6,8 +6,8 @@ norms around them are RMS norms on their results. The embedding is scaled.
 config.json keys read here:
   architecture "Mezadra"; vocab, width; norm.eps; embedding.scale (absent: 1);
   layers[i]: type ("attention" | "lightning"), mixer {...},
-    attention mixer: heads, kv_heads, dim, vdim, scale, conv (taps; absent: no convolution), rot {dims, base} (absent: no rotation),
-                     softcap (absent: none), v_mix (absent: false);
+    attention mixer: heads, kv_heads, dim, vdim, scale, conv (taps; absent or 0: no convolution), rot {dims, base} (absent: no
+                     rotation), softcap (absent or 0: none), v_mix (absent: false);
     lightning mixer: heads, dim, vdim, decay [one per head];
     mlp ({kind "dense", ff, limit} | {kind "moe", expert {ff}, router {experts, top}, shared {ff} (absent: none)} | null).
 Tensor names: embed, head, final.norm, l<i>.{norm1,norm2}, l<i>.mix.{q,k,v,o,sink,q.conv,k.conv,v.conv,vmix} or
@@ -78,9 +78,9 @@ class MezadraConfig:
                 if heads % kv:
                     raise ConfigError(f"config.json: '{mw}heads' {heads} is no multiple of kv_heads {kv}")
                 fields.update(scale=_get(m, "scale", mw, float), v_mix=bool(m.get("v_mix", False)))
-                if m.get("conv") is not None:
+                if m.get("conv"):
                     fields.update(conv=_get(m, "conv", mw, int, True))
-                if m.get("softcap") is not None:
+                if m.get("softcap"):
                     fields.update(softcap=_get(m, "softcap", mw, float, True))
                 if m.get("rot"):
                     dims = _get(m["rot"], "dims", mw + "rot.", int)

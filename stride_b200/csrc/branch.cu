@@ -61,7 +61,7 @@ __device__ __forceinline__ float mul(float a, float c) { return __fmul_rn(a, c);
 __device__ __forceinline__ float4 mul(float4 a, float c) { return make_float4(__fmul_rn(a.x, c), __fmul_rn(a.y, c), __fmul_rn(a.z, c), __fmul_rn(a.w, c)); }
 __device__ __forceinline__ float4 mul(float4 a, float4 c) { return make_float4(__fmul_rn(a.x, c.x), __fmul_rn(a.y, c.y), __fmul_rn(a.z, c.z), __fmul_rn(a.w, c.w)); }
 
-template <class V, bool CLEAR = true>
+template <class V, bool CLEAR = true, int IN_FLIGHT = kInFlight>
 __device__ __forceinline__ V source_value(const Source& s, int64_t i) {      // i in units of V
   V v = zero_of<V>();
   if (s.h != nullptr) {
@@ -72,15 +72,15 @@ __device__ __forceinline__ V source_value(const Source& s, int64_t i) {      // 
   if (s.partials != nullptr && s.n_partials > 0) {
     const V* p = reinterpret_cast<const V*>(s.partials) + i;
     const int64_t stride = s.stride / static_cast<int64_t>(sizeof(V) / sizeof(float));
-    V part[kInFlight];
+    V part[IN_FLIGHT];
 #pragma unroll
-    for (int k = 0; k < kInFlight; ++k)
+    for (int k = 0; k < IN_FLIGHT; ++k)
       if (k < s.n_partials) part[k] = p[k * stride];
     V sum = part[0];
 #pragma unroll
-    for (int k = 1; k < kInFlight; ++k)
+    for (int k = 1; k < IN_FLIGHT; ++k)
       if (k < s.n_partials) sum = add(sum, part[k]);
-    for (int k = kInFlight; k < s.n_partials; ++k) sum = add(sum, p[k * stride]);
+    for (int k = IN_FLIGHT; k < s.n_partials; ++k) sum = add(sum, p[k * stride]);
     v = s.h != nullptr ? add(v, sum) : sum;
   }
   return v;
@@ -134,9 +134,10 @@ __global__ void __launch_bounds__(256) branch_fold_kernel(float* __restrict__ ds
 // A block per row: the row's values (the branches read and cleared as above) stay in shared memory between the sum of squares and the
 // scaled add. The squares are added by a thread in ascending columns, then over the block in `block_sum`'s order. VEC: the width is a
 // multiple of four and every buffer 16-byte aligned: four elements a thread and request. Which form runs depends on the width and the
-// buffers alone, never on the rows of the step.
-template <class TG, bool VEC>
-__global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict__ dst, Source a, Source b, const TG* __restrict__ gain, int W,
+// buffers alone, never on the rows of the step; how many partial sums are requested together (IN_FLIGHT; one where there is no more than
+// one of either branch, which leaves registers for more blocks an SM) changes no addition.
+template <class TG, bool VEC, int IN_FLIGHT>
+__global__ void __launch_bounds__(256, IN_FLIGHT == 1 ? 4 : 2) branch_norm_fold_kernel(float* __restrict__ dst, Source a, Source b, const TG* __restrict__ gain, int W,
                                                                float eps, bf16* __restrict__ copy) {
   extern __shared__ __align__(16) float row_values[];
   __shared__ float red[32];
@@ -150,8 +151,8 @@ __global__ void __launch_bounds__(256) branch_norm_fold_kernel(float* __restrict
     float4* held = reinterpret_cast<float4*>(row_values);
     for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
       const int64_t i = (row + c) / 4;
-      float4 v = mul(source_value<float4, false>(a, i), ca);       // (cleared below: a store here would hold up the next requests)
-      if (two) v = add(v, mul(source_value<float4, false>(b, i), cb));
+      float4 v = mul(source_value<float4, false, IN_FLIGHT>(a, i), ca);       // (cleared below: a store here would hold up the next requests)
+      if (two) v = add(v, mul(source_value<float4, false, IN_FLIGHT>(b, i), cb));
       held[c / 4] = v;
       sq = fmaf(v.x, v.x, sq), sq = fmaf(v.y, v.y, sq), sq = fmaf(v.z, v.z, sq), sq = fmaf(v.w, v.w, sq);
     }
@@ -255,10 +256,15 @@ SB_EXPORT int sb_branch_norm_fold_ex(float* dst, float* a, const float* pa, int 
   const bool vec = W % 4 == 0 && aligned16(dst) && aligned16(a) && aligned16(pa) && aligned16(b) && aligned16(pb) && aligned16(gain) &&
                    sa % 4 == 0 && sb_ % 4 == 0 && aligned16(copy);
   const int threads = W >= 1024 ? 256 : 128;
-#define SB_NORM_FOLD(TG, VEC)                                                                                                              \
+#define SB_NORM_FOLD(TG, VEC)                             \
+  do {                                                    \
+    if (A.n_partials <= 1 && B.n_partials <= 1) SB_NORM_FOLD_P(TG, VEC, 1); \
+    else SB_NORM_FOLD_P(TG, VEC, kInFlight);              \
+  } while (0)
+#define SB_NORM_FOLD_P(TG, VEC, N)                                                                                                         \
   do {                                                                                                                                     \
-    if (smem > 48 * 1024) cudaFuncSetAttribute(branch_norm_fold_kernel<TG, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
-    sb::launch_pdl(branch_norm_fold_kernel<TG, VEC>, dim3(n), dim3(threads), smem, stream, dst, A, B, static_cast<const TG*>(gain), W, eps, \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(branch_norm_fold_kernel<TG, VEC, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
+    sb::launch_pdl(branch_norm_fold_kernel<TG, VEC, N>, dim3(n), dim3(threads), smem, stream, dst, A, B, static_cast<const TG*>(gain), W, eps, \
                    static_cast<bf16*>(copy));                                                                                              \
   } while (0)
   if (gain == nullptr || gain_dtype == 0) {
@@ -271,6 +277,7 @@ SB_EXPORT int sb_branch_norm_fold_ex(float* dst, float* a, const float* pa, int 
     return sb::fail("sb_branch_norm_fold: unsupported gain dtype %d", gain_dtype);
   }
 #undef SB_NORM_FOLD
+#undef SB_NORM_FOLD_P
   return sb::check_launch("sb_branch_norm_fold");
 }
 

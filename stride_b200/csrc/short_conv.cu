@@ -9,7 +9,7 @@
 // q is stored, k and v are appended to the token's pages. All of it is 32-bit. The last K - 1 inputs of a request, [K - 1][C] float32,
 // oldest first, are its record; where the sequence starts in the step nothing of the record is read. A token's result has the same bits
 // however the sequence was cut into steps: its inputs are the same sums wherever they come from, the taps are added oldest first, and a
-// head's squares are added by lane over fixed elements and then by xor shuffles.
+// head's squares are added by lane over fixed elements and then by xor shuffles (which elements, the sizes alone decide).
 #include "common.cuh"
 #include "step_ops.h"
 
@@ -78,20 +78,20 @@ struct ConvParams {
   int Hq, Hkv, D, Dv;
 };
 
-// A block per (tile of an entry's tokens, head of q, k or v). The tile's inputs and the taps - 1 in front of it wait in shared memory, then a
+// The general form: any sizes, any number of taps. A block per (tile of an entry's tokens, head of q, k or v). The tile's inputs and the taps - 1 in front of it wait in shared memory, then a
 // warp takes a token at a time. The block of an entry's first tile is the only one that touches the request's record: it reads what it
 // needs of it first and writes the new one, its columns of it, when it is done.
 template <class T, bool VEC>
 __global__ void __launch_bounds__(128) conv_qkv_kernel(ConvParams p) {
   extern __shared__ __align__(16) float smem[];
   sb::grid_launch_dependents();
-  const int unit = blockIdx.y, halo = p.taps - 1;
+  const int unit = blockIdx.y, taps = p.taps, halo = taps - 1;
   const bool is_q = unit < p.Hq, is_v = unit >= p.Hq + p.Hkv;
   const int head = is_q ? unit : is_v ? unit - p.Hq - p.Hkv : unit - p.Hq;
   const int nq = p.Hq * p.D, nk = p.Hkv * p.D, C = nq + nk + p.Hkv * p.Dv;
   const int dim = is_v ? p.Dv : p.D, c0 = is_q ? head * p.D : is_v ? nq + nk + head * p.Dv : nq + head * p.D;
   float* w = smem;                                   // [taps][dim]
-  float* in = w + p.taps * dim;                      // [halo + tile][dim]: row i is position first + i - halo
+  float* in = w + taps * dim;                      // [halo + tile][dim]: row i is position first + i - halo
   float* out = in + (halo + p.tile) * dim;           // [tile][dim]
   int e = 0, tile = blockIdx.x, len = 1;
   if (p.tile == 1) {
@@ -110,7 +110,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(ConvParams p) {
   constexpr int VE = VEC ? 4 : 1;
   const int per = dim / VE;
   if (p.conv != nullptr)
-    for (int i = threadIdx.x; i < p.taps * dim; i += blockDim.x) w[i] = p.conv[static_cast<int64_t>(i / dim) * C + c0 + i % dim];
+    for (int i = threadIdx.x; i < taps * dim; i += blockDim.x) w[i] = p.conv[static_cast<int64_t>(i / dim) * C + c0 + i % dim];
   float* record = p.record != nullptr ? p.record + static_cast<int64_t>(slot) * p.record_size + c0 : nullptr;
   sb::grid_dependency_wait();
   for (int i = threadIdx.x; i < (halo + nt) * per; i += blockDim.x) {
@@ -146,7 +146,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(ConvParams p) {
     auto convolved = [&](int d) {
       if (p.conv == nullptr) return u[d + halo * dim];
       float acc = 0.0f;
-      for (int j = 0; j < p.taps; ++j) acc = fmaf(w[j * dim + d], u[j * dim + d], acc);
+      for (int j = 0; j < taps; ++j) acc = fmaf(w[j * dim + d], u[j * dim + d], acc);
       return acc;
     };
     const int row = row0 + t0 + t, pos = pos0 + t0 + t;
@@ -190,6 +190,159 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(ConvParams p) {
   }
 }
 
+// The form for two to four taps and heads of up to 128 elements, in fours: L lanes (a power of two) own a head of q, k or v, four elements
+// each, and walk kRun consecutive tokens of an entry with the last inputs in registers: nothing passes through shared memory. The lanes of an
+// entry's first run read and write the request's record, each its own columns of it.
+constexpr int kRun = 8;
+
+__device__ __forceinline__ float4 fma4(float4 w, float4 u, float4 acc) {
+  return make_float4(fmaf(w.x, u.x, acc.x), fmaf(w.y, u.y, acc.y), fmaf(w.z, u.z, acc.z), fmaf(w.w, u.w, acc.w));
+}
+__device__ __forceinline__ void store4(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store4(bf16* dst, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 packed;
+  packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+  packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(dst) = packed;
+}
+
+// ONE: the projection left one buffer (long steps), nothing is folded.
+template <class T, int TAPS, bool ONE>
+__global__ void __launch_bounds__(128) conv_qkv_run_kernel(ConvParams p, int L) {
+  constexpr int HALO = TAPS - 1;
+  sb::grid_launch_dependents();
+  const int lane = threadIdx.x & (L - 1), units = p.Hq + 2 * p.Hkv;
+  const int unit = min(static_cast<int>(blockIdx.y) * (128 / L) + static_cast<int>(threadIdx.x) / L, units - 1);     // (surplus lanes repeat the
+  const bool real = static_cast<int>(blockIdx.y) * (128 / L) + static_cast<int>(threadIdx.x) / L < units;            //  last unit, storing nothing)
+  const bool is_q = unit < p.Hq, is_v = unit >= p.Hq + p.Hkv;
+  const int head = is_q ? unit : is_v ? unit - p.Hq - p.Hkv : unit - p.Hq;
+  const int nq = p.Hq * p.D, nk = p.Hkv * p.D, C = nq + nk + p.Hkv * p.Dv;
+  const int dim = is_v ? p.Dv : p.D, d = lane * 4;
+  const bool mine = d < dim, stores = mine && real;
+  const int c = (is_q ? head * p.D : is_v ? nq + nk + head * p.Dv : nq + head * p.D) + (mine ? d : 0);
+  int e = 0, run = blockIdx.x, len = 1;
+  if (p.tile == 1) {
+    e = run, run = 0;
+  } else {
+    for (; e < p.entries; ++e) {
+      len = p.meta[2 * p.meta_stride + e];
+      const int runs = (len + kRun - 1) / kRun;
+      if (run < runs) break;
+      run -= runs;
+    }
+  }
+  if (e >= p.entries) return;
+  const int slot = p.meta[e], row0 = p.meta[p.meta_stride + e], pos0 = p.meta[3 * p.meta_stride + e];
+  const int t0 = run * kRun, nt = min(kRun, len - t0);
+  const int rh = p.rot / 2;
+  const bool turned = !is_v && d < p.rot, low = d < rh;
+  const int partner = turned ? (low ? lane + rh / 4 : lane - rh / 4) : lane, pair = low ? d : d - rh;
+  const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  float4 w[TAPS], u[TAPS];                          // u: the inputs of the token and of those in front of it, oldest first
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) w[j] = *reinterpret_cast<const float4*>(p.conv + static_cast<int64_t>(j) * C + c);
+  float* record = p.record + static_cast<int64_t>(slot) * p.record_size + c;
+  const float* src = p.proj + static_cast<int64_t>(row0) * p.width + c;
+  sb::grid_dependency_wait();
+  auto input = [&](int t) {
+    const float* at = src + static_cast<int64_t>(t) * p.width;
+    return ONE ? *reinterpret_cast<const float4*>(at) : folded4(at, p.n_partials, p.partial_stride);
+  };
+  float4 last[HALO];                                // the inputs in front of the run
+#pragma unroll
+  for (int j = 0; j < HALO; ++j) {
+    const int t = t0 - HALO + j;
+    last[j] = t >= 0 ? input(t) : pos0 + t >= 0 ? *reinterpret_cast<const float4*>(record + static_cast<int64_t>(HALO + t) * C) : zero;
+  }
+  float4 first_inputs[HALO];
+#pragma unroll
+  for (int j = 0; j < HALO; ++j) first_inputs[j] = u[j + 1] = last[j];
+  constexpr int kAhead = ONE ? 4 : 1;               // tokens whose inputs are requested together
+  for (int t1 = 0; t1 < nt; t1 += kAhead) {
+    float4 next[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+      if (t1 + i < nt) next[i] = input(t0 + t1 + i);
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      if (t1 + i >= nt) break;
+      const int row = row0 + t0 + t1 + i, pos = pos0 + t0 + t1 + i;
+#pragma unroll
+      for (int j = 0; j < HALO; ++j) u[j] = u[j + 1];
+      u[HALO] = next[i];
+      float4 y = zero;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) y = fma4(w[j], u[j], y);
+      if (!mine) y = zero;
+      // (the lanes of v and of elements that are not turned take part in the exchange and leave its result)
+      const float4 b = make_float4(__shfl_sync(0xffffffffu, y.x, partner, L), __shfl_sync(0xffffffffu, y.y, partner, L),
+                                   __shfl_sync(0xffffffffu, y.z, partner, L), __shfl_sync(0xffffffffu, y.w, partner, L));
+      if (turned) {
+        const float4* cs = reinterpret_cast<const float4*>(p.cos_sin + (static_cast<int64_t>(pos) * rh + pair) * 2);
+        const float4 c01 = cs[0], c23 = cs[1];       // cos, sin of pairs 0 and 1; of pairs 2 and 3
+        auto turn = [&](float a, float o, float cs_, float sn) {
+          return low ? __fsub_rn(__fmul_rn(a, cs_), __fmul_rn(o, sn)) : __fadd_rn(__fmul_rn(a, cs_), __fmul_rn(o, sn));
+        };
+        y = make_float4(turn(y.x, b.x, c01.x, c01.y), turn(y.y, b.y, c01.z, c01.w), turn(y.z, b.z, c23.x, c23.y), turn(y.w, b.w, c23.z, c23.w));
+      }
+      if (p.unit) {
+        float ss = fmaf(y.w, y.w, fmaf(y.z, y.z, fmaf(y.y, y.y, __fmul_rn(y.x, y.x))));
+        for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o, L);
+        const float scale = is_v ? 1.0f : 1.0f / sqrtf(ss / static_cast<float>(dim) + p.eps);
+        y = make_float4(__fmul_rn(y.x, scale), __fmul_rn(y.y, scale), __fmul_rn(y.z, scale), __fmul_rn(y.w, scale));
+      }
+      if (!stores) continue;
+      if (is_q) {
+        store4(static_cast<T*>(p.q_out) + static_cast<int64_t>(row) * nq + c, y);
+        continue;
+      }
+      if (is_v && p.mix != kOwn) {
+        float* kept = p.kept + static_cast<int64_t>(row) * p.Hkv * p.Dv + head * p.Dv + d;
+        if (p.mix == kKeep) {
+          store4(kept, y);
+        } else {
+          const float4 k = *reinterpret_cast<const float4*>(kept);
+          y = make_float4(fmaf(p.lambda, k.x, __fmul_rn(p.rest, y.x)), fmaf(p.lambda, k.y, __fmul_rn(p.rest, y.y)),
+                          fmaf(p.lambda, k.z, __fmul_rn(p.rest, y.z)), fmaf(p.lambda, k.w, __fmul_rn(p.rest, y.w)));
+        }
+      }
+      const int page = p.block_table[static_cast<int64_t>(slot) * p.max_pages + pos / p.page_size];
+      store4(static_cast<T*>(p.pages) + static_cast<int64_t>(page) * p.page_stride + (is_v ? p.v_offset : 0) + static_cast<int64_t>(head) * p.head_stride +
+                 static_cast<int64_t>(pos % p.page_size) * p.Dc + d, y);
+    }
+  }
+  if (t0 != 0 || !stores) return;
+#pragma unroll
+  for (int j = 0; j < HALO; ++j) {                  // the record behind the step: its row j is the entry's token len - HALO + j
+    const int t = len - HALO + j;
+    float4 v = zero;
+    if (t >= 0) {
+      v = input(t);
+    } else {                                        // (a step shorter than the record: t = -1 is the newest of the inputs in front of it)
+#pragma unroll
+      for (int k = 0; k < HALO; ++k)
+        if (k == HALO + t) v = first_inputs[k];
+    }
+    *reinterpret_cast<float4*>(record + static_cast<int64_t>(j) * C) = v;
+  }
+}
+
+template <class T>
+void launch_run(const ConvParams& p, int n, int L, cudaStream_t stream) {
+  const int groups = 128 / L, units = p.Hq + 2 * p.Hkv;
+  const dim3 grid(p.tile == 1 ? p.entries : (n + kRun - 1) / kRun + p.entries, (units + groups - 1) / groups);
+#define SB_RUN(N)                                                                                                   \
+  do {                                                                                                              \
+    if (p.n_partials == 1) sb::launch_pdl(conv_qkv_run_kernel<T, N, true>, grid, dim3(128), 0, stream, p, L);       \
+    else sb::launch_pdl(conv_qkv_run_kernel<T, N, false>, grid, dim3(128), 0, stream, p, L);                        \
+  } while (0)
+  if (p.taps == 4) SB_RUN(4);
+  else if (p.taps == 3) SB_RUN(3);
+  else SB_RUN(2);
+#undef SB_RUN
+}
+
 }  // namespace
 
 // i: 0 projection partial sums (flat), 1 their width, 2 K ranges S, 3 most tokens with a buffer per range, 4 the taps [taps][C] (0: no
@@ -226,8 +379,18 @@ SB_EXPORT int sb_op_conv_qkv(const SbOp* op, const SbStep* s, void* stream) {
   const size_t smem = sizeof(float) * static_cast<size_t>(dim) * (p.taps + (p.taps - 1 + p.tile) + p.tile);
   if (smem > 200 * 1024) return sb::fail("sb_op_conv_qkv: heads of %d elements do not fit shared memory", dim), SB_OP_FAILED;
   const bool vec = p.D % 4 == 0 && p.Dv % 4 == 0 && p.width % 4 == 0 && p.record_size % 4 == 0 && ((op->i[0] | op->i[6]) & 15) == 0;
-  const dim3 grid(p.tile == 1 ? p.entries : (n + kTile - 1) / kTile + p.entries, p.Hq + 2 * p.Hkv), block(p.tile == 1 ? 64 : 128);
+  if (dtype != 0 && dtype != 1) return sb::fail("sb_op_conv_qkv: unsupported dtype %d", dtype), SB_OP_FAILED;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  // (which form runs depends on the sizes and the buffers alone, never on the rows of the step)
+  if (vec && p.taps >= 2 && p.taps <= 4 && dim <= 128 && p.rot % 8 == 0 && p.Dc % 4 == 0 && p.page_stride % 4 == 0 && p.v_offset % 4 == 0 &&
+      p.head_stride % 4 == 0 && ((op->i[4] | op->i[8] | op->i[11] | op->i[13] | op->i[15]) & 15) == 0) {
+    int L = 1;
+    while (L * 4 < dim) L *= 2;
+    if (dtype == 0) launch_run<float>(p, n, L, st);
+    else launch_run<bf16>(p, n, L, st);
+    return sb::check_launch("sb_op_conv_qkv");
+  }
+  const dim3 grid(p.tile == 1 ? p.entries : (n + kTile - 1) / kTile + p.entries, p.Hq + 2 * p.Hkv), block(p.tile == 1 ? 64 : 128);
 #define SB_CONV(T, V)                                                                                                            \
   do {                                                                                                                           \
     if (smem > 48 * 1024) cudaFuncSetAttribute(conv_qkv_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
@@ -235,9 +398,8 @@ SB_EXPORT int sb_op_conv_qkv(const SbOp* op, const SbStep* s, void* stream) {
   } while (0)
   if (dtype == 0 && vec) SB_CONV(float, true);
   else if (dtype == 0) SB_CONV(float, false);
-  else if (dtype == 1 && vec) SB_CONV(bf16, true);
-  else if (dtype == 1) SB_CONV(bf16, false);
-  else return sb::fail("sb_op_conv_qkv: unsupported dtype %d", dtype), SB_OP_FAILED;
+  else if (vec) SB_CONV(bf16, true);
+  else SB_CONV(bf16, false);
 #undef SB_CONV
   return sb::check_launch("sb_op_conv_qkv");
 }

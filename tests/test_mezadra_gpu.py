@@ -162,7 +162,8 @@ def _cache(part, slots, per, page, dtype, g):
     (4, 2, 22, 27, 60, 3, (10, 50.0), 1.5, 0.5, 8, torch.float32), (3, 3, 64, 64, 96, 4, (32, 1000.0), 4.0, 0.3, 16, torch.float32),
     (2, 1, 16, 40, 40, 0, None, 0.0, 0.4, 8, torch.float32),
     (8, 2, 64, 64, 128, 4, (32, 1000.0), 3.0, 0.15, 64, BF), (4, 4, 128, 128, 128, 3, (128, 500.0), 2.0, 0.1, 16, BF), (16, 1, 64, 64, 64, 2, None, 0.0, 0.1, 8, BF),
-    (6, 2, 64, 64, 72, 4, (8, 30.0), 5.0, 0.2, 24, BF), (4, 2, 48, 80, 96, 4, (48, 1000.0), 3.0, 0.2, 16, BF), (5, 5, 20, 12, 72, 2, (4, 9.0), 2.0, 0.5, 8, BF)])
+    (6, 2, 64, 64, 72, 4, (8, 30.0), 5.0, 0.2, 24, BF), (6, 2, 64, 64, 72, 4, (24, 30.0), 5.0, 0.2, 64, BF),
+    (12, 1, 128, 128, 64, 3, (16, 30.0), 4.0, 0.1, 32, BF), (12, 4, 64, 32, 64, 5, (12, 30.0), 3.0, 0.2, 32, BF), (4, 2, 48, 80, 96, 4, (48, 1000.0), 3.0, 0.2, 16, BF), (5, 5, 20, 12, 72, 2, (4, 9.0), 2.0, 0.5, 8, BF)])
 def test_attention_alone(H, G, D, V, W, taps, rot, cap, scale, page, dtype):
     """Two mixers, the second of which mixes its values with the first one's: two requests of unequal length fed in portions beside single
     tokens (long enough that a row's keys are folded over several chunks), in every attention kernel the shapes choose."""
