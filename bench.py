@@ -403,7 +403,7 @@ def _mezadra_config(width: int, ff: int, vocab: int, pairs: int, dense: bool = F
     """`pairs` times (attention behind a short convolution, lightning), heads as in the Keralorn configuration; the attention layers have a
     clamped dense feed-forward, the lightning layers eight experts of ff / 4, one per token, and a gated shared one (`dense`: all are dense)."""
     att = {"type": "attention", "mlp": {"kind": "dense", "ff": ff, "limit": 7.0},
-           "mixer": {"heads": width // 64, "kv_heads": width // 256, "dim": 64, "vdim": 64, "scale": 0.125, "conv": 4, "softcap": 30.0, "v_mix": True,
+           "mixer": {"heads": width // 64, "kv_heads": width // 256, "dim": 64, "vdim": 64, "scale": 0.125, "conv": 4, "softcap": 20.0, "v_mix": True,
                      "rot": {"dims": 32, "base": 500000.0}}}
     heads = width // 128
     moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 8, "top": 1}, "shared": {"ff": ff // 4}}
@@ -1107,7 +1107,7 @@ def _mezadra_kernels(timed, pk: dict, width: int, ff: int) -> dict:
         out = torch.empty(n, H * D, dtype=bf, device=dev)
         plan = program.plan(H // G, 128, 1, -1)
         keys = sum(past + t + 1 for t in range(length)) * entries
-        for name, floats, extra in (("attention_capped_with_sinks_", [0.125, 30.0], sinks), ("keralorn_attention_", [0.125, 0.0], None)):
+        for name, floats, extra in (("attention_capped_with_sinks_", [0.125, 20.0], sinks), ("keralorn_attention_", [0.125, 0.0], None)):
             if length > 1:
                 ms = timed(op("attention_tc5", "sb_op_attention_tc5", [q, out, pages, pages.shape[0], *where[1:], H, G, D, 0, plan, extra], floats), 5, clear=True)
                 record(name + label, ms, None, 4.0 * keys * H * D)

@@ -591,7 +591,7 @@ def test_long_decoding_and_slot_reuse(dtype, mezadra_dirs):
         eng.cache.check()
 
 
-def test_a_far_token_shows(mezadra_dirs, tmp_path):
+def test_a_far_token_shows(tmp_path):
     """Another token near the start moves the plain logits 300 tokens later far beyond the tolerance; the engine, fed in portions that cut
     pages and then token by token, agrees."""
     from stride_b200.engine.engine import StepEntry
